@@ -114,6 +114,15 @@ inline TqGlu tq_glu_params(float limit, float slope, float offset, int kind = TQ
     TqGlu p; p.limit = limit > 0.f ? limit : INFINITY; p.slope = slope; p.offset = offset; p.kind = kind; return p;
 }
 
+// Functions of one element (the Python side's MAP_* codes): the value itself, or the square of relu.
+#define TQ_MAP_COPY 0
+#define TQ_MAP_RELU_SQUARED 1
+inline bool tq_map_known(int map) { return map == TQ_MAP_COPY || map == TQ_MAP_RELU_SQUARED; }
+__device__ __forceinline__ float tq_map_element(float v, int map) {
+    if (map == TQ_MAP_RELU_SQUARED) { v = fmaxf(v, 0.f); v = v * v; }
+    return v;
+}
+
 // Element e of a head after the rotation of its first `dims` elements by the angles pos * freq[i] (float32):
 // pairs (2i, 2i+1) (halves == 0) or (i, i + dims/2) (halves != 0); the pair (u, v) becomes
 // (u cos - v sin, v cos + u sin).  Elements from `dims` on pass unchanged.  `head` holds the unrotated values.

@@ -544,8 +544,7 @@ __global__ void map_kernel(const TI* __restrict__ in, TO* __restrict__ out, size
     const size_t stride = (size_t)gridDim.x * blockDim.x;
     for (; i < n; i += stride) {
         float v = tq_to_float(in[i]);
-        if (act == 1) { v = fmaxf(v, 0.f); v = v * v; }
-        out[i] = tq_from_float<TO>(v);
+        out[i] = tq_from_float<TO>(tq_map_element(v, act));
     }
 }
 
@@ -826,22 +825,26 @@ TQ_EXPORT int tq_glu_table_rows(const float* z, const int* tokens, const void* t
 }
 
 // ---------------------------------------------------------------------------------------
-// x[t, j] = x[t, j] * scale + bias[j] for j < N, rows of `stride` floats (bias may be null).  Grid (row, column chunks).
+// x[t, j] = x[t, j] * scale + bias[j] for j < N, rows of `stride` floats (bias may be null), and with cap > 0 then
+// cap * tanh(x[t, j] / cap).  Grid (row, column chunks).
 // ---------------------------------------------------------------------------------------
-__global__ void scale_bias_cols_kernel(float* __restrict__ x, const float* __restrict__ bias, float scale, int N, int stride) {
+__global__ void scale_bias_cols_kernel(float* __restrict__ x, const float* __restrict__ bias, float scale, float cap, int N, int stride) {
     tq_grid_wait();                    // everything below may read what the previous kernel wrote
     tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
     float* row = x + (size_t)blockIdx.x * stride;
-    for (int j = blockIdx.y * blockDim.x + threadIdx.x; j < N; j += gridDim.y * blockDim.x)
-        row[j] = bias ? row[j] * scale + bias[j] : row[j] * scale;
+    for (int j = blockIdx.y * blockDim.x + threadIdx.x; j < N; j += gridDim.y * blockDim.x) {
+        const float v = bias ? row[j] * scale + bias[j] : row[j] * scale;
+        row[j] = cap > 0.f ? cap * tanhf(v / cap) : v;
+    }
 }
 
-TQ_EXPORT int tq_scale_bias_cols(float* x, const float* bias, float scale, int T_, int N, int stride, cudaStream_t stream) {
+TQ_EXPORT int tq_scale_bias_cols(float* x, const float* bias, float scale, float cap, int T_, int N, int stride, cudaStream_t stream) {
     if (T_ == 0) return 0;
+    TQ_REQUIRE(cap >= 0.f, "scale_bias_cols: a cap of %f", (double)cap);
     TQ_REQUIRE(N > 0 && N <= stride, "scale_bias_cols: %d columns of rows of %d", N, stride);
     // a few rows of many columns (a head's logits) spread over blocks by columns as well: 2048 columns a block
     const int threads = N >= 1024 ? 256 : 128;
-    tq_launch(dim3(T_, (N + 8 * threads - 1) / (8 * threads)), threads, 0, stream)(scale_bias_cols_kernel, x, bias, scale, N, stride);
+    tq_launch(dim3(T_, (N + 8 * threads - 1) / (8 * threads)), threads, 0, stream)(scale_bias_cols_kernel, x, bias, scale, cap, N, stride);
     TQ_CHECK_LAUNCH("scale_bias_cols");
     return 0;
 }
@@ -994,6 +997,140 @@ TQ_EXPORT int tq_dyt(float* x, const void* y, int y_dtype, float scale, const in
 }
 
 // ---------------------------------------------------------------------------------------
+// Two sub-layers that read the same norm, summed into the stream, with the norm that reads the stream next:
+//   x[r] += s1 * a[r] + s2 * b[r]        s1, s2: a factor per element (fp32 [H]; null: 1)
+//   out[q] = tanh(alpha * x[r]) * w + bias                              (no `out`: the sum alone)
+// b[r] is a row of its own (k == 0; b may be null) or the weighted sum of k rows of the expert-sorted layout,
+// sum_j wts[r, j] * b[row_of_pair[r * k + j]].  rows: only the norms of these rows are taken and x stays as it is; else
+// every row in order, and x takes its sum.  VEC neighbouring elements a thread (4: 16-byte accesses).  Grid
+// (rows, column chunks).
+// ---------------------------------------------------------------------------------------
+template <int VEC, typename T> __device__ __forceinline__ void load_vec(const T* p, float (&v)[VEC]) {
+    if constexpr (VEC == 4) { const float4 f = tq_load4<T>(p); v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
+    else v[0] = tq_to_float(*p);
+}
+template <int VEC, typename T> __device__ __forceinline__ void store_vec(T* p, const float (&v)[VEC]) {
+    if constexpr (VEC == 4) tq_store4<T>(p, make_float4(v[0], v[1], v[2], v[3]));
+    else *p = tq_from_float<T>(v[0]);
+}
+
+template <int VEC, typename TW, typename TO>
+__global__ void branches_dyt_kernel(float* __restrict__ x, const float* __restrict__ a, const float* __restrict__ s1,
+                                    const float* __restrict__ b, const float* __restrict__ s2, const int* __restrict__ row_of_pair,
+                                    const float* __restrict__ wts, int k, int b_rows, const int* __restrict__ rows, float alpha,
+                                    const TW* __restrict__ w, const TW* __restrict__ bias, TO* __restrict__ out, int H) {
+    tq_grid_wait();                    // everything below may read what the previous kernel wrote
+    tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
+    const size_t q = blockIdx.x;
+    const size_t r = rows ? (size_t)rows[q] : q;
+    for (int i = VEC * (blockIdx.y * blockDim.x + threadIdx.x); i < H; i += VEC * gridDim.y * blockDim.x) {
+        float v[VEC], f[VEC], t[VEC];
+        load_vec<VEC>(x + r * H + i, v);
+        load_vec<VEC>(a + r * H + i, f);
+        if (s1) {
+            load_vec<VEC>(s1 + i, t);
+#pragma unroll
+            for (int c = 0; c < VEC; ++c) f[c] *= t[c];
+        }
+        if (b) {
+            float g[VEC];
+            if (k == 0) {
+                load_vec<VEC>(b + r * H + i, g);
+            } else {
+#pragma unroll
+                for (int c = 0; c < VEC; ++c) g[c] = 0.f;
+#pragma unroll 4
+                for (int j = 0; j < k; ++j) {                   // unrolled: the chosen experts' rows load side by side
+                    const float wj = wts[r * k + j];
+                    load_vec<VEC>(b + (size_t)TQ_CHECKED(row_of_pair[r * k + j], b_rows, TQ_IDX_ROW) * H + i, t);
+#pragma unroll
+                    for (int c = 0; c < VEC; ++c) g[c] += wj * t[c];
+                }
+            }
+            if (s2) {
+                load_vec<VEC>(s2 + i, t);
+#pragma unroll
+                for (int c = 0; c < VEC; ++c) g[c] *= t[c];
+            }
+#pragma unroll
+            for (int c = 0; c < VEC; ++c) f[c] += g[c];
+        }
+#pragma unroll
+        for (int c = 0; c < VEC; ++c) v[c] += f[c];
+        if (rows == nullptr) store_vec<VEC>(x + r * H + i, v);
+        if (out != nullptr) {
+            float wi[VEC], bi[VEC];
+            load_vec<VEC>(w + i, wi);
+            load_vec<VEC>(bias + i, bi);
+#pragma unroll
+            for (int c = 0; c < VEC; ++c) v[c] = tanhf(alpha * v[c]) * wi[c] + bi[c];
+            store_vec<VEC>(out + q * H + i, v);
+        }
+    }
+}
+
+// R: rows taken; b_rows: rows of b (what row_of_pair is checked against in a debug build).
+TQ_EXPORT int tq_branches_dyt(float* x, const float* a, const float* s1, const float* b, const float* s2, const int* row_of_pair,
+                              const float* wts, int k, int b_rows, const int* rows, float alpha, const void* w, const void* bias,
+                              int w_dtype, void* out, int out_dtype, int R, int H, cudaStream_t stream) {
+    if (R == 0) return 0;
+    TQ_REQUIRE(H >= 1 && k >= 0 && a != nullptr, "branches: rows of %d elements, %d expert rows each", H, k);
+    TQ_REQUIRE(k == 0 || (b != nullptr && row_of_pair != nullptr && wts != nullptr), "branches: expert rows want their places and weights");
+    TQ_REQUIRE(out == nullptr || (w != nullptr && bias != nullptr), "branches: the norm wants its weight and bias");
+    TQ_REQUIRE(out != nullptr || rows == nullptr, "branches: chosen rows without a norm would do nothing");
+    auto aligned = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+    const bool vec = H % 4 == 0 && aligned(x) && aligned(a) && aligned(s1) && aligned(b) && aligned(s2) && aligned(w) &&
+                     aligned(bias) && aligned(out);
+    const int threads = H >= 1024 ? 256 : 128, per = (vec ? 4 : 1) * threads;
+    dim3 grid(R, (H + per - 1) / per);
+    TQ_REQUIRE(grid.y <= 65535, "branches: rows of %d elements exceed the grid limit", H);
+#define BRANCHES_LAUNCH(V)                                                                                              \
+    TQ_DISPATCH(w_dtype, TW, TQ_DISPATCH(out_dtype, TO,                                                                 \
+        (tq_launch(grid, threads, 0, stream)(branches_dyt_kernel<V, TW, TO>, x, a, s1, b, s2, row_of_pair, wts, k, b_rows, rows, \
+            alpha, (const TW*)w, (const TW*)bias, (TO*)out, H))))
+    if (vec) { BRANCHES_LAUNCH(4); } else { BRANCHES_LAUNCH(1); }
+#undef BRANCHES_LAUNCH
+    TQ_CHECK_LAUNCH("branches_dyt");
+    return 0;
+}
+
+// ---------------------------------------------------------------------------------------
+// x[t, j] = table[tokens[t], j] * scale + (j even: sin, odd: cos of 2 pi * positions[t] * turns[j / 2])
+// turns: a position's step in full turns per pair of columns, fp64 [(H + 1) / 2].  The turns are counted in fp64 and
+// only what is left of the last full one goes to fp32, so a far position's angle is as exact as a near one's.
+// ---------------------------------------------------------------------------------------
+template <typename TW>
+__global__ void embed_position_rows_kernel(const int* __restrict__ tokens, const int* __restrict__ positions,
+                                           const TW* __restrict__ table, const double* __restrict__ turns,
+                                           float* __restrict__ x, int H, int V, float scale) {
+    tq_grid_wait();                    // everything below may read what the previous kernel wrote
+    tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
+    const int t = blockIdx.x;
+    const TW* row = table + (size_t)TQ_CHECKED(tokens[t], V, TQ_IDX_TOKEN) * H;
+    const double p = (double)positions[t];
+    float* out = x + (size_t)t * H;
+    for (int m = blockIdx.y * blockDim.x + threadIdx.x; 2 * m < H; m += gridDim.y * blockDim.x) {
+        const double full = p * turns[m];
+        float sn, cs;
+        sincospif((float)(2.0 * (full - rint(full))), &sn, &cs);
+        out[2 * m] = tq_to_float(row[2 * m]) * scale + sn;
+        if (2 * m + 1 < H) out[2 * m + 1] = tq_to_float(row[2 * m + 1]) * scale + cs;
+    }
+}
+
+TQ_EXPORT int tq_embed_position_rows(const int* tokens, const int* positions, const void* table, int table_dtype, const double* turns,
+                                     float* x, int T_, int H, int V, float scale, cudaStream_t stream) {
+    if (T_ == 0) return 0;
+    TQ_REQUIRE(T_ > 0 && H > 0 && turns != nullptr, "embed_position_rows: bad sizes T=%d H=%d, or no table of turns", T_, H);
+    const int pairs = (H + 1) / 2, threads = pairs >= 512 ? 256 : 128;
+    TQ_DISPATCH(table_dtype, TW,
+        tq_launch(dim3(T_, (pairs + threads - 1) / threads), threads, 0, stream)(embed_position_rows_kernel<TW>, tokens, positions,
+            (const TW*)table, turns, x, H, V, scale));
+    TQ_CHECK_LAUNCH("embed_position_rows");
+    return 0;
+}
+
+// ---------------------------------------------------------------------------------------
 // A weighted sum over the depth of a model: hist holds the stream as every layer so far left it, [n][N] fp32.
 // Entry `at` is written first as x + scale * (f + bias) (f: a sub-layer's output still to be added, rows of H
 // elements; bias [H]; both may be null), then out = sum over j <= at of weights[j] * hist[j].  x and out may be
@@ -1044,8 +1181,7 @@ __global__ void bias_map_kernel(const float* __restrict__ in, const TW* __restri
     const size_t stride = (size_t)gridDim.x * blockDim.x;
     for (; i < n; i += stride) {
         float v = in[i] + tq_to_float(bias[i % N]);
-        if (act == 1) { v = fmaxf(v, 0.f); v = v * v; }
-        out[i] = tq_from_float<TO>(v);
+        out[i] = tq_from_float<TO>(tq_map_element(v, act));
     }
 }
 

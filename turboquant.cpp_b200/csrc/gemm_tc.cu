@@ -2,7 +2,7 @@
 // the accumulator in tensor memory: the expert products of the mixture-of-experts feed-forward
 // (routed experts and the shared expert), for prompts and for decoding.
 //
-//   out[row, n] = sum_k X[row, k] * W[g(row), n, k]          (plain)
+//   out[row, n] = f(sum_k X[row, k] * W[g(row), n, k])       (plain; f: nothing, or the square of relu)
 //   out[row, n] = silu(X.Wg[n]) * (X.Wu[n])                   (SwiGLU: W holds gate rows [0, N) and
 //                                                              up rows [N, 2N) of each group)
 // as the reference's expert loop computes them on the CPU (src/engine/tq_moe.c:975-999: g = Wg x,
@@ -307,7 +307,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                const __grid_constant__ CUtensorMap map_x_tail, TO* __restrict__ out,
                const int* __restrict__ tile_expert, const int* __restrict__ tile_row0,
                const int* __restrict__ tile_count, const int* __restrict__ n_tiles, int R, int N, int K,
-               int stream_weights, int* __restrict__ status, int k_splits, TqGlu act, const __grid_constant__ SECOND second) {
+               int stream_weights, int* __restrict__ status, int k_splits, TqGlu act, int map, const __grid_constant__ SECOND second) {
     // Bit 1 of stream_weights: the weights, the tile list and the sizes were final before the kernel ahead of this
     // one in the stream started (a down projection behind its gate/up product; a product with one group), so the
     // thread that streams the weights does not wait for that kernel: its loads are in flight while the kernel ahead
@@ -596,7 +596,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                 } else if (n < Nn) {
 #pragma unroll
                     for (int j = 0; j < 16; ++j)
-                        if (c0 + j < t.count) out_u[(size_t)(t.row0 + c0 + j) * Nn + n] = tq_from_float<TO>(__uint_as_float(g[j]));
+                        if (c0 + j < t.count) out_u[(size_t)(t.row0 + c0 + j) * Nn + n] = tq_from_float<TO>(tq_map_element(__uint_as_float(g[j]), map));
                 }
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -672,7 +672,7 @@ template <int BN, bool SWIGLU, typename TO, bool PAIR, bool KSPLIT = false, type
 int launch(const CUtensorMap& mw, const CUtensorMap& mx, const CUtensorMap& mxt, void* out, const int* te, const int* tr,
            const int* tc, const int* nt, int grid_y, int R, int N, int K, int G, int* status, int sm_share_pct,
            int k_splits, cudaStream_t stream, const SECOND& second = SECOND(), long long tiles2 = 0, int early_weights = 0,
-           TqGlu act = TqGlu{INFINITY, 1.0f, 0.0f}) {
+           TqGlu act = TqGlu{INFINITY, 1.0f, 0.0f}, int map = TQ_MAP_COPY) {
     using T = Tile<BN, PAIR>;
     auto kern = gemm_tc_kernel<BN, SWIGLU, TO, PAIR, KSPLIT, SECOND>;
     static bool configured = false;
@@ -714,7 +714,7 @@ int launch(const CUtensorMap& mw, const CUtensorMap& mx, const CUtensorMap& mxt,
     const int grid = (int)(want < room ? want : room);
     tq_launch(grid, T::THREADS, T::SMEM_BYTES, stream, PAIR ? 2 : 1)(kern, mw, mx, mxt, (TO*)out, te, tr, tc, nt, R, N, K,
         /* stream_weights: on average at most one token tile per group */ ((te != nullptr && (long long)R <= (long long)G * BN) ? 1 : 0) | (early_weights ? 2 : 0), status,
-        k_splits, act, second);
+        k_splits, act, map, second);
     TQ_CHECK_LAUNCH("gemm_tc");
     return 0;
 }
@@ -733,14 +733,17 @@ int launch(const CUtensorMap& mw, const CUtensorMap& mx, const CUtensorMap& mxt,
 // partial sums over the s-th share of K; the caller adds them up.  early_weights: the caller vouches that W, the
 // tile arrays and n_tiles were final before the kernel ahead of this one in the stream started; the weight stream then
 // starts without waiting for that kernel (programmatic dependent launch), the token rows wait for it as always.
+// map: a function of each output element of a plain product (TQ_MAP_*).
 TQ_EXPORT int tq_gemm_tc(const void* X, const void* W, void* out, int out_dtype, const int* tile_expert,
                          const int* tile_row0, const int* tile_count, const int* n_tiles, int max_tiles, int bn,
                          int R, int N, int K, int G, int swiglu, int pair, int* status, int sm_share_pct,
-                         int k_splits, int early_weights, float glu_limit, float glu_slope, float glu_offset,
+                         int k_splits, int early_weights, float glu_limit, float glu_slope, float glu_offset, int map,
                          cudaStream_t stream) {
     if (R == 0 || (tile_expert && max_tiles == 0)) return 0;
     const TqGlu act = tq_glu_params(glu_limit, glu_slope, glu_offset);       // (0, 1, 0): silu(gate) * up
     TQ_REQUIRE(k_splits >= 1, "gemm_tc: %d shares of K", k_splits);
+    TQ_REQUIRE(tq_map_known(map) && !((swiglu || k_splits > 1) && map != TQ_MAP_COPY),
+               "gemm_tc: element function %d (plain products with K in one piece only)", map);
     if (k_splits > 1) {
         TQ_REQUIRE(!swiglu && out_dtype == TQ_F32, "gemm_tc: K is shared out only for plain products with float32 partial sums");
         const int num_kb = (K + BK - 1) / BK, per = (num_kb + k_splits - 1) / k_splits;
@@ -762,7 +765,7 @@ TQ_EXPORT int tq_gemm_tc(const void* X, const void* W, void* out, int out_dtype,
     if (rc) return rc;
     rc = make_map_x(&mxt, X, (uint64_t)K, (uint64_t)R, 16u);
     if (rc) return rc;
-#define TC_ARGS mw, mx, mxt, out, tile_expert, tile_row0, tile_count, n_tiles, grid_y, R, N, K, G, status, sm_share_pct, k_splits, stream, NoSecond(), 0, early_weights, act
+#define TC_ARGS mw, mx, mxt, out, tile_expert, tile_row0, tile_count, n_tiles, grid_y, R, N, K, G, status, sm_share_pct, k_splits, stream, NoSecond(), 0, early_weights, act, map
 #define TC_CASE(BN_, PAIR_)                                                                          \
     if (bn == BN_ && (pair != 0) == PAIR_) {                                                         \
         if (swiglu) {                                                                                \
@@ -805,7 +808,7 @@ TQ_EXPORT int tq_gemm_tc_dual(const void* X, const void* W, void* out, const int
     TQ_REQUIRE((swiglu && out_dtype == TQ_BF16) || (!swiglu && out_dtype == TQ_F32),
                "gemm_tc_dual: SwiGLU products write bfloat16 and plain products float32 (got swiglu=%d, type %d)", swiglu, out_dtype);
     TQ_REQUIRE(status != nullptr, "gemm_tc_dual: a status word is required");
-    if (max_tiles == 0) return tq_gemm_tc(X2, W2, out2, out_dtype, nullptr, nullptr, nullptr, nullptr, 0, bn, R2, N2, K2, 1, swiglu, 1, status, 0, 1, 0, glu_limit2, glu_slope, glu_offset, stream);
+    if (max_tiles == 0) return tq_gemm_tc(X2, W2, out2, out_dtype, nullptr, nullptr, nullptr, nullptr, 0, bn, R2, N2, K2, 1, swiglu, 1, status, 0, 1, 0, glu_limit2, glu_slope, glu_offset, TQ_MAP_COPY, stream);
     const int cols = swiglu ? BM / 2 : BM;
     const int n_m1 = (N + cols - 1) / cols, n_m1_2 = (N2 + cols - 1) / cols;
     CUtensorMap mw, mx, mxt;

@@ -274,32 +274,48 @@ TQ_EXPORT int tq_router_select(float* logits, int* ids, float* wts, float* share
     return 0;
 }
 
-// The selection for one row by one warp (see router_select_corrected_kernel): row: E logits; c: E floats and gb:
-// n_groups floats of scratch (global or shared memory).
-__device__ __forceinline__ void select_corrected_row(const float* row, const float* __restrict__ correction, float* c,
-                                                     float* gb, int* __restrict__ ids_row, float* __restrict__ wts_row,
-                                                     int E, int k, int renorm, float floor_, int n_groups,
-                                                     int keep_groups, int lane) {
-    float mx = -INFINITY;
-    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, row[e]);
-    mx = tq_warp_max(mx);
-    float sum = 0.f;
-    for (int e = lane; e < E; e += 32) sum += expf(row[e] - mx);
-    sum = tq_warp_sum(sum);
-    for (int e = lane; e < E; e += 32) c[e] = expf(row[e] - mx) / sum + (correction ? correction[e] : 0.f);
+// How a selection that looks at more than the k largest logits chooses (see router_select_corrected_kernel).
+struct TqChoice {
+    const float* correction;     // one number per expert, added to the scores for the choice only (or null)
+    int active;                  // 0: the plain selection (softmax, k largest logits); the rest is then unused
+    float floor_;                // added to the chosen scores' sum before the division
+    int n_groups, keep_groups;   // equal groups of neighbouring experts, and how many of them may be chosen from
+    int group_top;               // a group's value: the sum of its group_top (1 or 2) largest choice values
+    int sigmoid;                 // the scores: sigmoid of each logit by itself (1), or the softmax over all (0)
+};
+
+// The selection for one row by one warp: row: E logits; c: E floats and gb: n_groups floats of scratch (global or
+// shared memory).  picks: where the choices go besides ids_row (shared memory of the caller), or null.
+__device__ __forceinline__ void select_corrected_row(const float* row, const TqChoice& how, float* c, float* gb,
+                                                     int* __restrict__ ids_row, float* __restrict__ wts_row, int E, int k,
+                                                     int renorm, int lane, int* picks) {
+    float mx = 0.f, sum = 1.f;
+    if (!how.sigmoid) {
+        mx = -INFINITY;
+        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, row[e]);
+        mx = tq_warp_max(mx);
+        sum = 0.f;
+        for (int e = lane; e < E; e += 32) sum += expf(row[e] - mx);
+        sum = tq_warp_sum(sum);
+    }
+    auto score = [&](int e) { return how.sigmoid ? 1.0f / (1.0f + expf(-row[e])) : expf(row[e] - mx) / sum; };
+    for (int e = lane; e < E; e += 32) c[e] = score(e) + (how.correction ? how.correction[e] : 0.f);
     __syncwarp();
-    if (n_groups > 1) {
-        const int per = E / n_groups;
-        for (int g = lane; g < n_groups; g += 32) {
-            float b = -INFINITY;
-            for (int e = g * per; e < (g + 1) * per; ++e) b = fmaxf(b, c[e]);
-            gb[g] = b;
+    if (how.n_groups > 1) {
+        const int per = E / how.n_groups;
+        for (int g = lane; g < how.n_groups; g += 32) {
+            float b = -INFINITY, b2 = -INFINITY;
+            for (int e = g * per; e < (g + 1) * per; ++e) {
+                const float v = c[e];
+                if (v > b) { b2 = b; b = v; } else if (v > b2) { b2 = v; }
+            }
+            gb[g] = how.group_top > 1 && per > 1 ? b + b2 : b;
         }
         __syncwarp();
-        for (int j = 0; j < keep_groups; ++j) {          // the kept groups are marked with +inf
+        for (int j = 0; j < how.keep_groups; ++j) {      // the kept groups are marked with +inf
             float best = -INFINITY;
             int best_g = 0x7fffffff;
-            for (int g = lane; g < n_groups; g += 32) {
+            for (int g = lane; g < how.n_groups; g += 32) {
                 const float v = gb[g];
                 if (v != INFINITY && (v > best || (v == best && g < best_g) || best_g == 0x7fffffff) && v == v) { best = v; best_g = g; }
             }
@@ -317,72 +333,85 @@ __device__ __forceinline__ void select_corrected_row(const float* row, const flo
     }
     float picked_sum = 0.f;
     for (int j = 0; j < k; ++j) {
-        float best = -INFINITY;
+        unsigned best = 0;
         int best_e = 0x7fffffff;
         for (int e = lane; e < E; e += 32) {
-            const float v = c[e];
-            if (v > best || (v == best && e < best_e)) { best = v; best_e = e; }   // NaN and minus infinity never win
+            const unsigned key = tq_order_key(c[e]);
+            if (key > best) { best = key; best_e = e; }                            // NaN and minus infinity never win
         }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-            const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
-            if (ov > best || (ov == best && oe < best_e)) { best = ov; best_e = oe; }
-        }
-        const bool found = best_e != 0x7fffffff && best != -INFINITY;
-        if (!found) best_e = j;                  // nothing left that may be chosen: keep indices valid, weight 0
-        const float p = found ? expf(row[best_e] - mx) / sum : 0.f;
+        const unsigned top = __reduce_max_sync(0xffffffffu, best);
+        int pick = __reduce_min_sync(0xffffffffu, (best == top && top != 0u) ? best_e : 0x7fffffff);
+        const bool found = pick != 0x7fffffff;
+        if (!found) pick = j;                    // nothing left that may be chosen: keep indices valid, weight 0
+        const float p = found ? score(pick) : 0.f;
         picked_sum += p;                         // identical in every lane
         if (lane == 0) {
-            ids_row[j] = best_e;
+            ids_row[j] = pick;
             wts_row[j] = p;
-            if (found) c[best_e] = -INFINITY;
+            if (picks) picks[j] = pick;
+            if (found) c[pick] = -INFINITY;
         }
         __syncwarp();
     }
     if (renorm) {
         __syncwarp();
-        for (int j = lane; j < k; j += 32) wts_row[j] = wts_row[j] / (picked_sum + floor_);
+        for (int j = lane; j < k; j += 32) wts_row[j] = wts_row[j] / (picked_sum + how.floor_);
     }
 }
 
-// Selection with a correction of the choice and groups of experts, one warp per token.  s = softmax(logits) over all
-// E experts; the choice looks at c = s + correction (correction may be null: c = s); with n_groups > 1 the experts form
-// n_groups equal groups of neighbours, a group's value is its largest c, and only experts of the keep_groups groups
-// with the largest values can be chosen (the others count as minus infinity); the k largest c are chosen (ties to
-// the lowest index); the weights are the chosen experts' s, divided by (their sum + floor) if renorm.
-// choice: T * E floats of scratch; group_best: T * n_groups floats of scratch (n_groups > 1).
-__global__ void router_select_corrected_kernel(const float* __restrict__ logits, const float* __restrict__ correction,
-                                               float* __restrict__ choice, float* __restrict__ group_best,
-                                               int* __restrict__ ids, float* __restrict__ wts,
-                                               float* __restrict__ shared_scale, int T_, int E, int k, int renorm,
-                                               float floor_, int n_groups, int keep_groups) {
+// Selection with other scores, a correction of the choice and groups of experts, one warp per token.  s = softmax of
+// the logits over all E experts, or each logit's sigmoid; the choice looks at c = s + correction (correction may be
+// null: c = s); with n_groups > 1 the experts form n_groups equal groups of neighbours, a group's value is the sum of
+// its one or two largest c, and only experts of the keep_groups groups with the largest values can be chosen (the
+// others count as minus infinity); the k largest c are chosen (ties to the lowest index); the weights are the chosen
+// experts' s, divided by (their sum + floor) if renorm.
+// choice: T * E floats of scratch and group_best: T * n_groups floats (n_groups > 1), or both null: the warps' rows
+// of scratch, E + n_groups floats each, are then in dynamic shared memory.
+__global__ void router_select_corrected_kernel(const float* __restrict__ logits, float* __restrict__ choice,
+                                               float* __restrict__ group_best, int* __restrict__ ids, float* __restrict__ wts,
+                                               float* __restrict__ shared_scale, int T_, int E, int k, int renorm, TqChoice how) {
     tq_grid_wait();                    // everything below may read what the previous kernel wrote
     tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
+    extern __shared__ float s_choice[];
     const int lane = threadIdx.x & 31;
     const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (t >= T_) return;
     const float* row = logits + (size_t)t * (E + 1);
-    float* c = choice + (size_t)t * E;
+    float* c = choice ? choice + (size_t)t * E : s_choice + (size_t)(threadIdx.x >> 5) * (E + how.n_groups);
+    float* gb = choice ? (group_best ? group_best + (size_t)t * how.n_groups : nullptr) : c + E;
     if (shared_scale && lane == 0) shared_scale[t] = 1.0f / (1.0f + expf(-row[E]));
-    select_corrected_row(row, correction, c, group_best ? group_best + (size_t)t * n_groups : nullptr, ids + (size_t)t * k,
-                         wts + (size_t)t * k, E, k, renorm, floor_, n_groups, keep_groups, lane);
+    select_corrected_row(row, how, c, gb, ids + (size_t)t * k, wts + (size_t)t * k, E, k, renorm, lane, nullptr);
 }
+
+// What every launcher of this selection checks.
+static int check_choice(const TqChoice& how, int E, int k) {
+    TQ_REQUIRE(how.n_groups >= 1 && E % how.n_groups == 0, "router: %d experts do not form %d equal groups", E, how.n_groups);
+    TQ_REQUIRE(how.n_groups == 1 || (how.keep_groups >= 1 && how.keep_groups <= how.n_groups), "router: %d of %d groups kept",
+               how.keep_groups, how.n_groups);
+    TQ_REQUIRE(how.n_groups == 1 || how.keep_groups * (E / how.n_groups) >= k, "router: %d groups of %d experts cannot give %d choices",
+               how.keep_groups, E / how.n_groups, k);
+    TQ_REQUIRE(how.group_top == 1 || how.group_top == 2, "router: a group's value from its %d largest scores (1 or 2 are known)",
+               how.group_top);
+    return 0;
+}
+
+// E + n_groups up to this many: a warp's scratch of the selection fits shared memory (four warps a block)
+#define SELECT_SHARED_FLOATS 2560
 
 TQ_EXPORT int tq_router_select_corrected(const float* logits, const float* correction, float* choice, float* group_best,
                                          int* ids, float* wts, float* shared_scale, int T_, int E, int k, int renorm,
-                                         float floor_, int n_groups, int keep_groups, cudaStream_t stream) {
+                                         float floor_, int n_groups, int keep_groups, int group_top, int sigmoid,
+                                         cudaStream_t stream) {
     if (T_ == 0) return 0;
     TQ_REQUIRE(E >= 1 && E <= ROUTER_MAX_EXPERTS, "router: %d experts exceed %d", E, ROUTER_MAX_EXPERTS);
     TQ_REQUIRE(k >= 1 && k <= E, "router: top-k %d must be in 1..%d", k, E);
-    TQ_REQUIRE(choice != nullptr, "router: scratch for the choice values is required");
-    TQ_REQUIRE(n_groups >= 1 && E % n_groups == 0, "router: %d experts do not form %d equal groups", E, n_groups);
-    TQ_REQUIRE(n_groups == 1 || (keep_groups >= 1 && keep_groups <= n_groups && group_best != nullptr),
-               "router: %d of %d groups kept", keep_groups, n_groups);
-    TQ_REQUIRE(n_groups == 1 || keep_groups * (E / n_groups) >= k, "router: %d groups of %d experts cannot give %d choices",
-               keep_groups, E / n_groups, k);
-    tq_launch((T_ + 3) / 4, 128, 0, stream)(router_select_corrected_kernel, logits, correction, choice, group_best, ids, wts,
-                                            shared_scale, T_, E, k, renorm, floor_, n_groups, keep_groups);
+    const TqChoice how = {correction, 1, floor_, n_groups, keep_groups, group_top, sigmoid};
+    if (int rc = check_choice(how, E, k)) return rc;
+    TQ_REQUIRE(choice == nullptr || n_groups == 1 || group_best != nullptr, "router: scratch for the groups' values is required");
+    TQ_REQUIRE(choice != nullptr || E + n_groups <= SELECT_SHARED_FLOATS, "router: scratch for the choice values is required");
+    const size_t smem = choice == nullptr ? (size_t)4 * (E + n_groups) * sizeof(float) : 0;
+    tq_launch((T_ + 3) / 4, 128, smem, stream)(router_select_corrected_kernel, logits, choice, group_best, ids, wts,
+                                               shared_scale, T_, E, k, renorm, how);
     TQ_CHECK_LAUNCH("router_select_corrected");
     return 0;
 }
@@ -645,6 +674,10 @@ __device__ __forceinline__ void small_layout(SmallShared& S, int P, int E, int k
 }
 
 // ---- the cluster form ----
+// bytes ahead of the rows in a block's dynamic shared memory: the logits, and the choice's scratch where it needs one
+__host__ __device__ __forceinline__ size_t small_front_bytes(int E, const TqChoice& how) {
+    return ((size_t)(E + 1 + (how.active ? E + how.n_groups : 0)) * 4 + 15) & ~(size_t)15;
+}
 __device__ __forceinline__ unsigned small_cluster_rank() { unsigned r; asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r)); return r; }
 __device__ __forceinline__ void small_cluster_sync() {
     asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
@@ -672,7 +705,7 @@ router_cluster_kernel(const TA* __restrict__ x, const TW* __restrict__ wr, const
                       int* __restrict__ counts, int* __restrict__ sorted_pair, int* __restrict__ row_of_pair,
                       int* __restrict__ expert_offset, int* __restrict__ tile_expert, int* __restrict__ tile_row0,
                       int* __restrict__ tile_count, int* __restrict__ n_tiles, TA* __restrict__ x_rows, int vec_x,
-                      const float* __restrict__ logit_bias) {
+                      const float* __restrict__ logit_bias, TqChoice how) {
     const unsigned rank = small_cluster_rank();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
     // a block's shared memory may be written by its peers only once it runs: every block says so here and
@@ -695,7 +728,8 @@ router_cluster_kernel(const TA* __restrict__ x, const TW* __restrict__ wr, const
     tq_grid_launch_dependents();
     extern __shared__ __align__(16) unsigned char s_raw[];
     float* s_logit = reinterpret_cast<float*>(s_raw);                         // [E + 1] the logits of this block's token
-    TA* s_x = reinterpret_cast<TA*>(s_raw + (((size_t)(E + 1) * 4 + 15) & ~(size_t)15));   // [T][H] the step's rows
+    float* s_choice = s_logit + E + 1;                                        // [E + groups] scratch of the choice, where it needs one
+    TA* s_x = reinterpret_cast<TA*>(s_raw + small_front_bytes(E, how));       // [T][H] the step's rows
     __shared__ SmallShared S;
     const TA* xs = tq_fresh(x);                                               // loads of x stay behind the wait
     if (vec_x) {
@@ -742,7 +776,10 @@ router_cluster_kernel(const TA* __restrict__ x, const TW* __restrict__ wr, const
     const int t = (int)rank;
     if (t < T_ && warp == 0) {
         if (shared_scale && lane == 0) shared_scale[t] = 1.0f / (1.0f + expf(-s_logit[E]));
-        select_in_registers(s_logit, E, k, renorm, lane, ids + (size_t)t * k, wts + (size_t)t * k, S.mine);
+        if (how.active)
+            select_corrected_row(s_logit, how, s_choice, s_choice + E, ids + (size_t)t * k, wts + (size_t)t * k, E, k, renorm, lane, S.mine);
+        else
+            select_in_registers(s_logit, E, k, renorm, lane, ids + (size_t)t * k, wts + (size_t)t * k, S.mine);
     }
     small_cluster_sync();                                     // every token's choices are in its block
     const int P = T_ * k;
@@ -796,7 +833,7 @@ router_tiny_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __r
                    int renorm, int* __restrict__ counts, int* __restrict__ sorted_pair, int* __restrict__ row_of_pair,
                    int* __restrict__ expert_offset, int* __restrict__ tile_expert, int* __restrict__ tile_row0,
                    int* __restrict__ tile_count, int* __restrict__ n_tiles, __nv_bfloat16* __restrict__ x_rows,
-                   const float* __restrict__ logit_bias) {
+                   const float* __restrict__ logit_bias, TqChoice how) {
     extern __shared__ __align__(16) unsigned char s_tiny[];
     __nv_bfloat16* s_x = reinterpret_cast<__nv_bfloat16*>(s_tiny);                     // [T][H]
     float* s_logit = reinterpret_cast<float*>(s_tiny + (size_t)T * H * 2);             // [T][E + 1]
@@ -861,7 +898,12 @@ router_tiny_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __r
     if (warp < T) {
         const float* row = s_logit + warp * (E + 1);
         if (shared_scale && lane == 0) shared_scale[warp] = 1.0f / (1.0f + expf(-row[E]));
-        select_in_registers(row, E, k, renorm, lane, ids + (size_t)warp * k, wts + (size_t)warp * k, s_ids + warp * k);
+        if (how.active) {
+            float* c = s_logit + T * (E + 1) + warp * (E + how.n_groups);        // this token's scratch of the choice
+            select_corrected_row(row, how, c, c + E, ids + (size_t)warp * k, wts + (size_t)warp * k, E, k, renorm, lane, s_ids + warp * k);
+        } else {
+            select_in_registers(row, E, k, renorm, lane, ids + (size_t)warp * k, wts + (size_t)warp * k, s_ids + warp * k);
+        }
     }
     __syncthreads();
     // ---- layout by counting ----
@@ -912,8 +954,7 @@ router_small_kernel(const TA* __restrict__ x, const TW* __restrict__ wr, const T
                     int* __restrict__ counts, int* __restrict__ sorted_pair, int* __restrict__ row_of_pair,
                     int* __restrict__ expert_offset, int* __restrict__ tile_expert, int* __restrict__ tile_row0,
                     int* __restrict__ tile_count, int* __restrict__ n_tiles, TA* __restrict__ x_rows, int vec_x,
-                    int* __restrict__ counter, const float* __restrict__ correction, int corrected, float floor_,
-                    int n_groups, int keep_groups, const float* __restrict__ logit_bias) {
+                    int* __restrict__ counter, TqChoice how, const float* __restrict__ logit_bias) {
     tq_grid_wait();
     tq_grid_launch_dependents();
     extern __shared__ float s_dyn[];
@@ -959,10 +1000,9 @@ router_small_kernel(const TA* __restrict__ x, const TW* __restrict__ wr, const T
     // ---- selection: warp 0 (the same choices and weights as router_select_kernel) ----
     if (warp == 0) {
         if (shared_scale && lane == 0) shared_scale[t] = 1.0f / (1.0f + expf(-s_logit[E]));
-        if (corrected) {
+        if (how.active) {
             // corrected scores and groups: the row's place (no longer needed) is the scratch, E + n_groups <= H floats
-            select_corrected_row(s_logit, correction, s_x, s_x + E, ids + (size_t)t * k, wts + (size_t)t * k, E, k, renorm,
-                                 floor_, n_groups, keep_groups, lane);
+            select_corrected_row(s_logit, how, s_x, s_x + E, ids + (size_t)t * k, wts + (size_t)t * k, E, k, renorm, lane, nullptr);
         } else if (E <= 32 * SELECT_REGS) {
             select_in_registers(s_logit, E, k, renorm, lane, ids + (size_t)t * k, wts + (size_t)t * k, nullptr);
         } else {
@@ -1052,13 +1092,12 @@ TQ_EXPORT int tq_router_small(const void* x, int act_dtype, const void* wr, cons
                               int* ids, float* wts, float* shared_scale, int tile_rows, int* counts, int* sorted_pair,
                               int* row_of_pair, int* expert_offset, int* tile_expert, int* tile_row0, int* tile_count,
                               int* n_tiles, void* x_rows, int* counter, int T_, int H, int E, int k, int renorm,
-                              const float* correction, int corrected, float floor_, int n_groups, int keep_groups,
-                              const float* logit_bias, cudaStream_t stream) {
+                              const float* correction, int corrected, float floor_, int n_groups, int keep_groups, int group_top,
+                              int sigmoid, const float* logit_bias, cudaStream_t stream) {
     if (T_ == 0) return 0;
-    if (corrected) {            // corrected scores, groups, a floor under the weights' sum: the counter form knows them
-        TQ_REQUIRE(n_groups >= 1 && E % n_groups == 0 && keep_groups >= 1 && keep_groups <= n_groups &&
-                   (n_groups == 1 || keep_groups * (E / n_groups) >= k), "router_small: %d of %d groups of %d experts for %d choices",
-                   keep_groups, n_groups, E / (n_groups > 0 ? n_groups : 1), k);
+    const TqChoice how = {correction, corrected, floor_, n_groups, keep_groups, group_top, sigmoid};
+    if (corrected) {            // other scores, a correction, groups, a floor under the weights' sum
+        if (int rc = check_choice(how, E, k)) return rc;
         TQ_REQUIRE(E + n_groups <= H, "router_small: %d experts and %d groups need scratch of a row of %d values", E, n_groups, H);
     }
     TQ_REQUIRE(T_ * k <= SMALL_MAX_PAIRS && E <= SMALL_MAX_EXPERTS,
@@ -1079,12 +1118,12 @@ TQ_EXPORT int tq_router_small(const void* x, int act_dtype, const void* wr, cons
     {
         const char* tiny_env = getenv("TQ_ROUTER_NO_TINY");
         const bool no_tiny = tiny_env && tiny_env[0] && tiny_env[0] != '0';
-        const size_t smem_tiny = (size_t)T_ * H * 2 + (size_t)T_ * (E + 1) * 4;
-        if (!corrected && !no_tiny && (T_ == 1 || (tiny_env && tiny_env[0] == '0' && T_ <= TINY_MAX_T)) && T_ * k <= TINY_MAX_PAIRS && T_ <= tile_rows && act_dtype == TQ_BF16 && w_dtype == TQ_BF16 &&
+        const size_t smem_tiny = (size_t)T_ * H * 2 + (size_t)T_ * (E + 1 + (corrected ? E + n_groups : 0)) * 4;
+        if (!no_tiny && (T_ == 1 || (tiny_env && tiny_env[0] == '0' && T_ <= TINY_MAX_T)) && T_ * k <= TINY_MAX_PAIRS && T_ <= tile_rows && act_dtype == TQ_BF16 && w_dtype == TQ_BF16 &&
             H % 8 == 0 && vec_w && vec_x && E <= 32 * SELECT_REGS && smem_tiny <= 40 * 1024) {
 #define TINY_CASE(TT) case TT: tq_launch(1, TINY_THREADS, smem_tiny, stream)(router_tiny_kernel<TT>, (const __nv_bfloat16*)x, \
             (const __nv_bfloat16*)wr, (const __nv_bfloat16*)wsg, ids, wts, shared_scale, H, E, k, renorm, counts, sorted_pair,  \
-            row_of_pair, expert_offset, tile_expert, tile_row0, tile_count, n_tiles, (__nv_bfloat16*)x_rows, logit_bias); break;
+            row_of_pair, expert_offset, tile_expert, tile_row0, tile_count, n_tiles, (__nv_bfloat16*)x_rows, logit_bias, how); break;
             switch (T_) { TINY_CASE(1) TINY_CASE(2) TINY_CASE(3) TINY_CASE(4) }
 #undef TINY_CASE
             TQ_CHECK_LAUNCH("router_tiny");
@@ -1092,9 +1131,9 @@ TQ_EXPORT int tq_router_small(const void* x, int act_dtype, const void* wr, cons
         }
     }
     // the cluster form (TQ_ROUTER_NO_CLUSTER=1: the counter form after all)
-    const size_t smem_cluster = (((size_t)(E + 1) * 4 + 15) & ~(size_t)15) + (size_t)T_ * H * abytes;
+    const size_t smem_cluster = small_front_bytes(E, how) + (size_t)T_ * H * abytes;
     const char* no_cluster = getenv("TQ_ROUTER_NO_CLUSTER");
-    const bool cluster = !corrected && T_ <= SMALL_CLUSTER && E <= 32 * SELECT_REGS && smem_cluster <= SMALL_CLUSTER_DYNAMIC_BYTES &&
+    const bool cluster = T_ <= SMALL_CLUSTER && E <= 32 * SELECT_REGS && smem_cluster <= SMALL_CLUSTER_DYNAMIC_BYTES &&
                          (vec_x || !vec_w) &&       // the order of a sum follows the weights' loads; the rows must allow the same
                          !(no_cluster && no_cluster[0] && no_cluster[0] != '0');
     if (cluster) {
@@ -1103,14 +1142,13 @@ TQ_EXPORT int tq_router_small(const void* x, int act_dtype, const void* wr, cons
         TQ_DISPATCH(act_dtype, TA, TQ_DISPATCH(w_dtype, TW,
             (cfg = launch_router_cluster<TA, TW>(smem_cluster, stream, (const TA*)x, (const TW*)wr, (const TW*)wsg,
                 ids, wts, shared_scale, T_, H, E, k, renorm, vec_dot, tile_rows, counts, sorted_pair, row_of_pair, expert_offset,
-                tile_expert, tile_row0, tile_count, n_tiles, (TA*)x_rows, vec_x, logit_bias))));
+                tile_expert, tile_row0, tile_count, n_tiles, (TA*)x_rows, vec_x, logit_bias, how))));
         TQ_REQUIRE(cfg == cudaSuccess, "router_small: %zu bytes of shared memory refused: %s", smem_cluster, cudaGetErrorString(cfg));
     } else {
         TQ_DISPATCH(act_dtype, TA, TQ_DISPATCH(w_dtype, TW,
             (tq_launch(T_, SMALL_THREADS, smem, stream)(router_small_kernel<TA, TW>, (const TA*)x, (const TW*)wr, (const TW*)wsg,
                 ids, wts, shared_scale, T_, H, E, k, renorm, vec_w, tile_rows, counts, sorted_pair, row_of_pair, expert_offset,
-                tile_expert, tile_row0, tile_count, n_tiles, (TA*)x_rows, vec_x, counter, correction, corrected, floor_,
-                n_groups, keep_groups, logit_bias))));
+                tile_expert, tile_row0, tile_count, n_tiles, (TA*)x_rows, vec_x, counter, how, logit_bias))));
     }
     TQ_CHECK_LAUNCH("router_small");
     return 0;
@@ -1132,7 +1170,7 @@ __global__ void __launch_bounds__(256)
 grouped_gemm_kernel(const TA* __restrict__ A, const TW* __restrict__ W, TO* __restrict__ C,
                     const int* __restrict__ tile_expert, const int* __restrict__ tile_row0,
                     const int* __restrict__ tile_count, const int* __restrict__ n_tiles,
-                    int R, int N, int K, TqGlu act) {
+                    int R, int N, int K, TqGlu act, int map) {
     tq_grid_wait();                    // everything below may read what the previous kernel wrote
     tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
     __shared__ float As[GG_BK][GG_BM + 4];
@@ -1209,7 +1247,7 @@ grouped_gemm_kernel(const TA* __restrict__ A, const TW* __restrict__ W, TO* __re
                 const float g = acc[0][i][j], u = acc[SWIGLU ? 1 : 0][i][j];
                 v = tq_glu(g, u, act);
             } else {
-                v = acc[0][i][j];
+                v = tq_map_element(acc[0][i][j], map);
             }
             C[(size_t)(row0 + r) * N + n] = tq_from_float<TO>(v);
         }
@@ -1247,7 +1285,7 @@ __global__ void __launch_bounds__(GV_WARPS * 32)
 grouped_gemv_kernel(const TA* __restrict__ A, const TW* __restrict__ W, TO* __restrict__ C,
                     const int* __restrict__ tile_expert, const int* __restrict__ tile_row0,
                     const int* __restrict__ tile_count, const int* __restrict__ n_tiles,
-                    int R, int N, int K, int tile_rows, int vec, TqGlu act) {
+                    int R, int N, int K, int tile_rows, int vec, TqGlu act, int map) {
     tq_grid_wait();                    // everything below may read what the previous kernel wrote
     tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
     extern __shared__ __align__(16) float s_rows[];          // [GV_ROWS][GV_KC]
@@ -1340,6 +1378,8 @@ grouped_gemv_kernel(const TA* __restrict__ A, const TW* __restrict__ W, TO* __re
                         if (SWIGLU) {
                             const float u = tq_warp_sum(acc[c][S - 1][r]);
                             v = tq_glu(v, u, act);
+                        } else {
+                            v = tq_map_element(v, map);
                         }
                         if (lane == 0) C[(size_t)(row0 + rb + r) * N + n] = tq_from_float<TO>(v);
                     }
@@ -1353,7 +1393,7 @@ grouped_gemv_kernel(const TA* __restrict__ A, const TW* __restrict__ W, TO* __re
 // tq_grouped_gemm.
 template <typename TA, typename TW, typename TO, bool SWIGLU>
 int launch_grouped_gemv(const void* A, const void* W, void* C, const int* te, const int* tr, const int* tc, const int* nt,
-                        int by, int R, int N, int K, int tile_rows, TqGlu act, cudaStream_t stream) {
+                        int by, int R, int N, int K, int tile_rows, TqGlu act, int map, cudaStream_t stream) {
     auto kern = grouped_gemv_kernel<TA, TW, TO, SWIGLU>;
     const int smem = GV_ROWS * GV_KC * (int)sizeof(float);
     static bool configured = false;
@@ -1366,16 +1406,17 @@ int launch_grouped_gemv(const void* A, const void* W, void* C, const int* te, co
     dim3 grid((N + cols - 1) / cols, by);
     // 16-byte (8-byte) loads of four weights: rows of K values that start on such a boundary
     const int vec = K % 4 == 0 && ((uintptr_t)W % (4 * sizeof(TW))) == 0;
-    tq_launch(grid, GV_WARPS * 32, smem, stream)(kern, (const TA*)A, (const TW*)W, (TO*)C, te, tr, tc, nt, R, N, K, tile_rows, vec, act);
+    tq_launch(grid, GV_WARPS * 32, smem, stream)(kern, (const TA*)A, (const TW*)W, (TO*)C, te, tr, tc, nt, R, N, K, tile_rows, vec, act, map);
     return 0;
 }
 
 TQ_EXPORT int tq_grouped_gemm(const void* A, int a_dtype, const void* W, int w_dtype, void* C, int c_dtype,
                               const int* tile_expert, const int* tile_row0, const int* tile_count,
                               const int* n_tiles, int max_tiles, int R, int N, int K, int swiglu, int few_rows,
-                              float glu_limit, float glu_slope, float glu_offset, cudaStream_t stream) {
+                              float glu_limit, float glu_slope, float glu_offset, int map, cudaStream_t stream) {
     if (R == 0 || (tile_expert && max_tiles == 0)) return 0;
     const TqGlu act = tq_glu_params(glu_limit, glu_slope, glu_offset);      // (0, 1, 0): silu(gate) * up
+    TQ_REQUIRE(tq_map_known(map) && !(swiglu && map != TQ_MAP_COPY), "grouped_gemm: element function %d (plain products only)", map);
     TQ_REQUIRE(R > 0 && N > 0 && K > 0, "grouped_gemm: bad sizes R=%d N=%d K=%d", R, N, K);
     const int by = tile_expert ? max_tiles : (R + GG_BM - 1) / GG_BM;
     TQ_REQUIRE(by <= 65535, "grouped_gemm: %d row tiles exceed the grid limit", by);
@@ -1386,8 +1427,8 @@ TQ_EXPORT int tq_grouped_gemm(const void* A, int a_dtype, const void* W, int w_d
     if (few_rows && gv_types) {
         int rc = 0;
 #define GV_LAUNCH(TA, TW, TO)                                                                                     \
-        rc = swiglu ? launch_grouped_gemv<TA, TW, TO, true>(A, W, C, tile_expert, tile_row0, tile_count, n_tiles, by, R, N, K, GG_BM, act, stream) \
-                    : launch_grouped_gemv<TA, TW, TO, false>(A, W, C, tile_expert, tile_row0, tile_count, n_tiles, by, R, N, K, GG_BM, act, stream)
+        rc = swiglu ? launch_grouped_gemv<TA, TW, TO, true>(A, W, C, tile_expert, tile_row0, tile_count, n_tiles, by, R, N, K, GG_BM, act, map, stream) \
+                    : launch_grouped_gemv<TA, TW, TO, false>(A, W, C, tile_expert, tile_row0, tile_count, n_tiles, by, R, N, K, GG_BM, act, map, stream)
         if (a_dtype == TQ_F32) GV_LAUNCH(float, float, float);
         else if (c_dtype == TQ_F32) GV_LAUNCH(__nv_bfloat16, __nv_bfloat16, float);
         else GV_LAUNCH(__nv_bfloat16, __nv_bfloat16, __nv_bfloat16);
@@ -1400,7 +1441,7 @@ TQ_EXPORT int tq_grouped_gemm(const void* A, int a_dtype, const void* W, int w_d
 #define GG_LAUNCH(SW)                                                                                   \
     TQ_DISPATCH(a_dtype, TA, TQ_DISPATCH(w_dtype, TW, TQ_DISPATCH(c_dtype, TO,                          \
         (tq_launch(grid, 256, 0, stream)(grouped_gemm_kernel<TA, TW, TO, SW>,                                  \
-            (const TA*)A, (const TW*)W, (TO*)C, tile_expert, tile_row0, tile_count, n_tiles, R, N, K, act)))))
+            (const TA*)A, (const TW*)W, (TO*)C, tile_expert, tile_row0, tile_count, n_tiles, R, N, K, act, map)))))
     if (swiglu) { GG_LAUNCH(true); } else { GG_LAUNCH(false); }
 #undef GG_LAUNCH
     TQ_CHECK_LAUNCH("grouped_gemm");

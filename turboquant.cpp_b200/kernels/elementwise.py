@@ -132,8 +132,9 @@ def glu_table_rows(z: torch.Tensor, tokens: torch.Tensor, table: torch.Tensor, c
 
 
 def scale_bias_cols(x: torch.Tensor, scale: float = 1.0, bias: Optional[torch.Tensor] = None,
-                    cols: Optional[int] = None) -> torch.Tensor:
-    """x[t, j] = x[t, j] * scale + bias[j] in place for the first `cols` columns (all by default) of float32 rows."""
+                    cols: Optional[int] = None, cap: float = 0.0) -> torch.Tensor:
+    """x[t, j] = x[t, j] * scale + bias[j] in place for the first `cols` columns (all by default) of float32 rows;
+    with cap > 0 then cap * tanh(x[t, j] / cap)."""
     want_f32(x, "the rows")
     T, S = x.shape
     N = S if cols is None else int(cols)
@@ -142,7 +143,8 @@ def scale_bias_cols(x: torch.Tensor, scale: float = 1.0, bias: Optional[torch.Te
         if bias.numel() != N:
             raise KernelError("scale_bias_cols: one bias per column")
     lib = load_kernel(_LIB)
-    check(_LIB, lib.tq_scale_bias_cols(ptr(x), ptr(bias), c_float(scale), c_int(T), c_int(N), c_int(S), stream()))
+    check(_LIB, lib.tq_scale_bias_cols(ptr(x), ptr(bias), c_float(scale), c_float(cap), c_int(T), c_int(N), c_int(S),
+                                      stream()))
     return x
 
 
@@ -293,6 +295,59 @@ def dyt(x: torch.Tensor, alpha: float, weight: torch.Tensor, bias: torch.Tensor,
                            c_longlong(state.stride(0) if state is not None else 0), ptr(seq_of_token), ptr(cu_seqlens),
                            ptr(slots), c_int(n_seqs), c_int(1 if single_tokens else 0), stream()),
           kernels=2 if shift is not None and not single_tokens else 1)
+    return out
+
+
+def branches_dyt(x: torch.Tensor, a: torch.Tensor, a_scale: Optional[torch.Tensor], b: Optional[torch.Tensor] = None,
+                 b_scale: Optional[torch.Tensor] = None, row_of_pair: Optional[torch.Tensor] = None,
+                 pair_weights: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, alpha: float = 1.0,
+                 weight: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
+                 out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x += a_scale * a + b_scale * b for the float32 rows of x [T, H] (the scales: float32 [H] or None), and
+    out = tanh(alpha * x) * weight + bias of the sum (out None: the sum alone).  b: [T, H], or with pair_weights
+    [T, k] the rows of an expert-sorted layout, of which token t's b is the sum over j of pair_weights[t, j] *
+    b[row_of_pair[t * k + j]].  rows: out[r] is the norm of row rows[r] and x is left alone."""
+    for t, what in ((x, "the residual stream"), (a, "the first branch"), (b, "the second branch"), (a_scale, "the first scale"),
+                    (b_scale, "the second scale"), (pair_weights, "the pairs' weights")):
+        if t is not None:
+            want_f32(t, what)
+    T, H = x.shape
+    k = 0
+    if pair_weights is not None:
+        want_int32(row_of_pair, "the pairs' rows")
+        k = pair_weights.shape[1]
+        if b is None or pair_weights.shape[0] != T or row_of_pair.numel() < T * k:
+            raise KernelError("branches_dyt: expert rows, their places and weights do not fit together")
+    if a.shape != x.shape or (b is not None and (b.shape[1] != H or (k == 0 and b.shape[0] != T))):
+        raise KernelError("branches_dyt: the branches do not have the stream's shape")
+    if any(s is not None and s.numel() != H for s in (a_scale, b_scale)):
+        raise KernelError("branches_dyt: one factor per element of the width")
+    if out is not None and (weight is None or bias is None or weight.dtype != bias.dtype):
+        raise KernelError("branches_dyt: the norm's weight and bias must share a dtype")
+    if rows is not None:
+        want_int32(rows, "rows")
+    R = T if rows is None else rows.shape[0]
+    lib = load_kernel(_LIB)
+    check(_LIB, lib.tq_branches_dyt(ptr(x), ptr(a), ptr(a_scale), ptr(b), ptr(b_scale), ptr(row_of_pair if k else None),
+                                    ptr(pair_weights), c_int(k), c_int(b.shape[0] if b is not None else 0), ptr(rows),
+                                    c_float(alpha), ptr(weight), ptr(bias), c_int(code(weight.dtype) if weight is not None else 0),
+                                    ptr(out), c_int(code(out.dtype) if out is not None else 0), c_int(R), c_int(H), stream()))
+    return x if out is None else out
+
+
+def embed_position_rows(tokens: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, turns: torch.Tensor, scale: float,
+                        out: torch.Tensor) -> torch.Tensor:
+    """out[t, j] = table[tokens[t], j] * scale + sin (even j) or cos (odd j) of 2 pi * positions[t] * turns[j // 2], as
+    float32.  turns float64 [(H + 1) // 2]: a position's step per pair of columns, in full turns."""
+    want_int32(tokens, "tokens")
+    want_int32(positions, "positions")
+    want_f32(out, "the residual stream")
+    T, H = out.shape
+    if turns.dtype != torch.float64 or turns.numel() != (H + 1) // 2:
+        raise KernelError("embed_position_rows: a float64 step per pair of columns")
+    lib = load_kernel(_LIB)
+    check(_LIB, lib.tq_embed_position_rows(ptr(tokens), ptr(positions), ptr(table), c_int(code(table.dtype)), ptr(turns), ptr(out),
+                                           c_int(T), c_int(H), c_int(table.shape[0]), c_float(scale), stream()))
     return out
 
 

@@ -129,7 +129,8 @@ _NO_PAIRS = os.environ.get("TQ_NO_PAIRS", "") not in ("", "0")
 
 def gemm_tc(x: torch.Tensor, w: PackedWeights, out: torch.Tensor, layout: Optional[ExpertLayout],
             token_tile: int, pair: Optional[bool] = None, status: Optional[torch.Tensor] = None,
-            sm_share: int = 0, k_splits: int = 1, early_weights: bool = False, glu=None) -> torch.Tensor:
+            sm_share: int = 0, k_splits: int = 1, early_weights: bool = False, glu=None,
+            map: int = 0) -> torch.Tensor:
     """x [R, K] bf16; w: packed weights of G groups; out [R, N] bf16 or fp32 (with w.swiglu:
     silu(x.Wg) * (x.Wu)).  layout: expert-sorted tiles of `token_tile` rows (None: one group).
     pair: run on pairs of CTAs (default: for wide token tiles, unless TQ_NO_PAIRS=1).  status: the int32 the
@@ -139,7 +140,8 @@ def gemm_tc(x: torch.Tensor, w: PackedWeights, out: torch.Tensor, layout: Option
     k_splits_for) and the caller adds the slices up in order.  early_weights: the caller vouches that the weights
     and the layout were final before the kernel ahead of this one in the stream started (a down projection behind
     its gate/up product); the kernel then starts streaming weights while that kernel still runs.
-    glu: the gated activation of a SwiGLU-packed product (kernels.elementwise.Glu; default silu(gate) * up)."""
+    glu: the gated activation of a SwiGLU-packed product (kernels.elementwise.Glu; default silu(gate) * up).  map: a
+    function of each output element of a plain product (kernels.elementwise.MAP_*)."""
     if pair is None:
         pair = token_tile >= PAIR_MIN_TILE and not _NO_PAIRS
     if not usable(x, w):
@@ -162,7 +164,7 @@ def gemm_tc(x: torch.Tensor, w: PackedWeights, out: torch.Tensor, layout: Option
         ptr(lo.n_tiles) if lo else None, c_int(lo.max_tiles if lo else 0), c_int(token_tile),
         c_int(R), c_int(N), c_int(K), c_int(w.groups), c_int(1 if w.swiglu else 0), c_int(1 if pair else 0),
         ptr(status if status is not None else status_word(x.device)), c_int(int(sm_share)), c_int(int(k_splits)),
-        c_int(1 if early_weights else 0), *_glu_args(glu), stream()))
+        c_int(1 if early_weights else 0), *_glu_args(glu), c_int(map), stream()))
     return out
 
 

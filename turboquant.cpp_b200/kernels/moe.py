@@ -72,11 +72,12 @@ def router_logits(x: torch.Tensor, w_router: torch.Tensor, w_shared_gate: Option
 
 def router_select_corrected(logits: torch.Tensor, correction: Optional[torch.Tensor], top_k: int, renorm: bool,
                             floor: float, n_groups: int, keep_groups: int, ids: torch.Tensor, weights: torch.Tensor,
-                            shared_scale: Optional[torch.Tensor]) -> None:
+                            shared_scale: Optional[torch.Tensor], sigmoid: bool = False, group_top: int = 1) -> None:
     """Selection on float32 logits [T, E + 1] with a correction of the choice and groups of experts: scores are the
-    softmax over all experts; the choice looks at score + correction [E] (float32, or None); with n_groups > 1 only
-    experts of the keep_groups groups (of E / n_groups neighbours) with the largest such value can be chosen; the
-    weights are the chosen experts' scores, divided by (their sum + floor) if renorm."""
+    softmax over all experts (sigmoid: each logit's sigmoid); the choice looks at score + correction [E] (float32, or
+    None); with n_groups > 1 only experts of the keep_groups groups (of E / n_groups neighbours) with the largest sum of
+    their group_top (1 or 2) largest such values can be chosen; the weights are the chosen experts' scores, divided by
+    (their sum + floor) if renorm."""
     want_f32(logits, "router logits")
     want_int32(ids, "expert ids")
     want_f32(weights, "expert weights")
@@ -84,13 +85,15 @@ def router_select_corrected(logits: torch.Tensor, correction: Optional[torch.Ten
         want_f32(correction, "the choice's correction")
     T, E1 = logits.shape
     E = E1 - 1
-    choice = torch.empty((T, E), dtype=torch.float32, device=logits.device)
-    group_best = torch.empty((T, n_groups), dtype=torch.float32, device=logits.device) if n_groups > 1 else None
+    choice = group_best = None             # the selection's scratch lies in shared memory where it fits
+    if E + n_groups > SELECT_SHARED_FLOATS:
+        choice = torch.empty((T, E), dtype=torch.float32, device=logits.device)
+        group_best = torch.empty((T, n_groups), dtype=torch.float32, device=logits.device) if n_groups > 1 else None
     lib = load_kernel(_LIB)
     check(_LIB, lib.tq_router_select_corrected(ptr(logits), ptr(correction), ptr(choice), ptr(group_best), ptr(ids),
                                                ptr(weights), ptr(shared_scale), c_int(T), c_int(E), c_int(top_k),
                                                c_int(1 if renorm else 0), c_float(floor), c_int(n_groups),
-                                               c_int(keep_groups), stream()))
+                                               c_int(keep_groups), c_int(group_top), c_int(1 if sigmoid else 0), stream()))
 
 
 def max_tiles(n_pairs: int, n_experts: int, tile_rows: int) -> int:
@@ -116,6 +119,7 @@ class ExpertLayout:
         self.chunk_hist = torch.empty(-(-max(1, n_pairs) // align_chunk(n_pairs)) * n_experts, **i32)     # scratch of moe_align
 
 
+SELECT_SHARED_FLOATS = 2560                           # csrc/moe.cu
 SMALL_MAX_PAIRS, SMALL_MAX_EXPERTS = 512, 1023      # what the kernel accepts
 SMALL_PAIRS_WORTH_IT = 128                           # beyond this one block is slower than the separate kernels
 
@@ -145,11 +149,11 @@ def router_small(x: torch.Tensor, w_router: torch.Tensor, w_shared_gate: Optiona
                  renorm: bool, ids: torch.Tensor, weights: torch.Tensor, shared_scale: Optional[torch.Tensor],
                  layout: ExpertLayout, x_rows: torch.Tensor, correction: Optional[torch.Tensor] = None,
                  corrected: bool = False, floor: float = 0.0, n_groups: int = 1, keep_groups: int = 1,
-                 logit_bias: Optional[torch.Tensor] = None) -> None:
+                 logit_bias: Optional[torch.Tensor] = None, sigmoid: bool = False, group_top: int = 1) -> None:
     """For steps of few tokens: router, expert-sorted layout and the sorted copies of the token rows
     (x_rows[row] = x[token of that row]) in one launch.  Launches on one device must not overlap (they share
     the counter that tells the last block its turn).  corrected: the selection of router_select_corrected
-    (correction [E] float32 or None, groups, floor); it needs n_experts + n_groups <= hidden.  logit_bias float32
+    (correction [E] float32 or None, groups, floor, sigmoid, group_top); it needs n_experts + n_groups <= hidden.  logit_bias float32
     [E]: added to the experts' logits before anything else looks at them."""
     if logit_bias is not None:
         want_f32(logit_bias, "the logits' bias")
@@ -167,7 +171,7 @@ def router_small(x: torch.Tensor, w_router: torch.Tensor, w_shared_gate: Optiona
         ptr(lo.row_of_pair), ptr(lo.expert_offset), ptr(lo.tile_expert), ptr(lo.tile_row0), ptr(lo.tile_count),
         ptr(lo.n_tiles), ptr(x_rows), ptr(_counter(x.device)), c_int(T), c_int(H), c_int(E), c_int(top_k),
         c_int(1 if renorm else 0), ptr(correction), c_int(1 if corrected else 0), c_float(floor), c_int(n_groups),
-        c_int(keep_groups), ptr(logit_bias), stream()))
+        c_int(keep_groups), c_int(group_top), c_int(1 if sigmoid else 0), ptr(logit_bias), stream()))
 
 
 def moe_align(ids: torch.Tensor, layout: ExpertLayout) -> None:
@@ -181,12 +185,13 @@ def moe_align(ids: torch.Tensor, layout: ExpertLayout) -> None:
 
 
 def grouped_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, layout: Optional[ExpertLayout],
-                 swiglu: bool, few_rows: bool = False, glu=None) -> torch.Tensor:
+                 swiglu: bool, few_rows: bool = False, glu=None, map: int = 0) -> torch.Tensor:
     """Exact (CUDA-core, fp32 accumulation) grouped product.  a [R, K]; w [G, Nw, K] with Nw = N,
     or 2N when swiglu (gate rows, then up rows); out [R, N].  layout None: one group (G = 1).
     few_rows: the tiles hold a few rows each (a decode step): the kernel that streams the weights once per eight
     rows of a tile instead of the tiled one (any number of rows is right, many are slow).
-    glu: the gated activation of a swiglu product (kernels.elementwise.Glu; default silu(gate) * up)."""
+    glu: the gated activation of a swiglu product (kernels.elementwise.Glu; default silu(gate) * up).  map: a
+    function of each output element of a plain product (kernels.elementwise.MAP_*)."""
     R, K = a.shape
     N = out.shape[1]
     if w.dim() == 2:
@@ -202,7 +207,7 @@ def grouped_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, layout: Op
         ptr(lo.tile_expert) if lo else None, ptr(lo.tile_row0) if lo else None,
         ptr(lo.tile_count) if lo else None, ptr(lo.n_tiles) if lo else None,
         c_int(lo.max_tiles if lo else 0), c_int(R), c_int(N), c_int(K), c_int(1 if swiglu else 0),
-        c_int(1 if few_rows else 0), c_float(g.limit), c_float(g.slope), c_float(g.offset), stream()))
+        c_int(1 if few_rows else 0), c_float(g.limit), c_float(g.slope), c_float(g.offset), c_int(map), stream()))
     return out
 
 

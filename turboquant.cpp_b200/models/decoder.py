@@ -11,6 +11,7 @@ step, with the LM head on the wanted rows only (the reference's multi-token path
 last row only, :3571-3587)."""
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 from typing import Dict, List, Optional, Sequence
 
@@ -98,12 +99,44 @@ class PairEmbedding(Embedding):
                                  None if last is None else last.view(-1), x)
 
 
+class PositionedEmbedding(Embedding):
+    """x = table[token] * scale + s(position): s interleaves sines and cosines, elements 2m and 2m + 1 being sin and cos
+    of position * base^(-2m / hidden).  The angles are counted in full turns in float64 (no longest position)."""
+
+    def __init__(self, name: str, vocab: int, hidden: int, scale: float = 1.0, base: float = 10000.0):
+        super().__init__(name, vocab, hidden)
+        if not base > 0.0:
+            raise ValueError(f"embedding '{name}': base {base} must be positive")
+        self.scale, self.base = float(scale), float(base)
+        self.turns: Optional[torch.Tensor] = None
+
+    def bind(self, store: WeightStore) -> None:
+        super().bind(store)
+        self.turns = position_turns(self.hidden, self.base).to(store.device)
+
+    def forward(self, tokens: torch.Tensor) -> torch.Tensor:
+        raise NotImplementedError("an embedding that looks at positions needs the step: use embed(ctx)")
+
+    def embed(self, ctx: StepContext) -> torch.Tensor:
+        x = torch.empty((ctx.tokens.shape[0], self.hidden), dtype=torch.float32, device=ctx.tokens.device)
+        return K.embed_position_rows(ctx.tokens, ctx.positions, self.table, self.turns, self.scale, x)
+
+
+def position_turns(hidden: int, base: float) -> torch.Tensor:
+    """base^(-2m / hidden) / (2 pi), float64, for every pair m of columns (the last one may be half a pair)."""
+    m = torch.arange((hidden + 1) // 2, dtype=torch.float64)
+    return torch.pow(torch.tensor(base, dtype=torch.float64), -2.0 * m / hidden) / (2.0 * math.pi)
+
+
 class LMHead(Part):
     """logits = W x in float32; ``name`` may be the embedding's tensor (tied weights:
-    src/engine/tq_model.c:1499-1516).  `scale`: a factor on the float32 logits."""
+    src/engine/tq_model.c:1499-1516).  `scale`: a factor on the float32 logits; `softcap` > 0: they then become
+    softcap * tanh(logits / softcap)."""
 
-    def __init__(self, name: str, vocab: int, hidden: int, scale: float = 1.0):
-        self.name, self.vocab, self.hidden, self.scale = name, int(vocab), int(hidden), float(scale)
+    def __init__(self, name: str, vocab: int, hidden: int, scale: float = 1.0, softcap: float = 0.0):
+        if softcap < 0.0:
+            raise ValueError(f"head '{name}': the cap {softcap} must not be negative")
+        self.name, self.vocab, self.hidden, self.scale, self.softcap = name, int(vocab), int(hidden), float(scale), float(softcap)
         self.weight: Optional[torch.Tensor] = None
 
     def weight_specs(self) -> List[WeightSpec]:
@@ -113,11 +146,13 @@ class LMHead(Part):
         self.weight = store.get(self.name)
 
     def kernels(self) -> List[str]:
-        return ["elementwise"] if self.scale != 1.0 else []
+        return ["elementwise"] if self.scale != 1.0 or self.softcap > 0.0 else []
 
     def forward(self, xn: torch.Tensor) -> torch.Tensor:
         logits = linear(xn, self.weight, out_dtype=torch.float32)
-        return logits if self.scale == 1.0 else K.scale_bias_cols(logits, self.scale)
+        if self.scale == 1.0 and self.softcap == 0.0:
+            return logits
+        return K.scale_bias_cols(logits, self.scale, cap=self.softcap)
 
     def step_work(self, n_tokens, kv_tokens):
         w = self.weight

@@ -1,5 +1,5 @@
 """Parts a model is put together from: norms, position encodings, mixers, feed-forwards, blocks."""
-from .base import (KVNeed, StateNeed, LayerCache, StepContext, Part, Norm, PositionEncoding, Mixer, FeedForward, Block,
+from .base import (ExpertRows, OpenSum, KVNeed, StateNeed, LayerCache, StepContext, Part, Norm, PositionEncoding, Mixer, FeedForward, Block,
                    register_mixer, register_feed_forward, register_norm, register_position_encoding,
                    make_mixer, make_feed_forward, make_norm, make_position_encoding,
                    MIXERS, FEED_FORWARDS, NORMS, POSITION_ENCODINGS)
@@ -16,4 +16,4 @@ from .parallel import ParallelMixer
 from .token_side import TokenSideInput
 from .dense_ffn import SwiGLUFeedForward, ReluSquaredFeedForward, GluFeedForward
 from .moe_ffn import MoEFeedForward
-from .block import PreNormBlock, PostNormBlock, SandwichBlock, DepthMixBlock
+from .block import PreNormBlock, PostNormBlock, SandwichBlock, DepthMixBlock, ParallelBlock

@@ -24,7 +24,8 @@ Mixer           cache_need() -> KVNeed | None; state_need() -> StateNeed | None;
 FeedForward     capturable() -> bool; forward(xn, ctx) -> y [T, hidden]
 Block           cache_need(); state_need(); capturable(); forward(x, pending, ctx, cache) -> (x, pending):
                 pending is a sub-layer output not yet added to the residual stream x (the sum is fused
-                into the next norm).  A model talks to its blocks only through this interface.
+                into the next norm), or an OpenSum of two of them.  A model talks to its blocks only through
+                this interface.
 
 capturable(): whether the part's forward can be recorded into a CUDA graph for decode steps: it reads
 everything that changes from step to step from device tensors of the StepContext (positions, slots, page
@@ -100,6 +101,37 @@ class StepContext:
     carry: Dict[str, torch.Tensor] = field(default_factory=dict)
 
 
+@dataclass
+class ExpertRows:
+    """A routed feed-forward's output before its last step: rows [T * k, H] float32 in the expert-sorted layout; token
+    t's output is the sum over j of weights[t, j] * rows[row_of_pair[t * k + j]]."""
+    rows: torch.Tensor
+    row_of_pair: torch.Tensor
+    weights: torch.Tensor
+
+
+@dataclass
+class OpenSum:
+    """What a block with two sub-layers under one norm leaves to be added to the stream: a_scale * a + b_scale * b, a
+    factor per element (float32 [H], or None for one); b is rows like a, ExpertRows, or None.  Only norms that say
+    `adds_open_sums` take one."""
+    a: torch.Tensor
+    a_scale: Optional[torch.Tensor]
+    b: Any = None
+    b_scale: Optional[torch.Tensor] = None
+
+    def operands(self) -> Dict[str, Any]:
+        """The arguments kernels.elementwise.branches_dyt takes for it."""
+        routed = isinstance(self.b, ExpertRows)
+        return dict(a=self.a, a_scale=self.a_scale, b=self.b.rows if routed else self.b, b_scale=self.b_scale,
+                    row_of_pair=self.b.row_of_pair if routed else None, pair_weights=self.b.weights if routed else None)
+
+    def float(self) -> torch.Tensor:
+        """The sum itself (for looking at the stream between layers; a step's own path never needs it)."""
+        from ..kernels.elementwise import branches_dyt
+        return branches_dyt(torch.zeros_like(self.a), **self.operands())
+
+
 class Part:
     def weight_specs(self) -> List[WeightSpec]:
         return []
@@ -120,6 +152,8 @@ class Part:
 
 
 class Norm(Part):
+    adds_open_sums = False        # whether `add` (forward) and `y` (add_forward) may be an OpenSum
+
     def forward(self, x: torch.Tensor, out_dtype: torch.dtype, rows: Optional[torch.Tensor] = None,
                 add: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Norm of the rows of x (of x + add if add is given); with `rows`, of those rows only.

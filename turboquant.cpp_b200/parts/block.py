@@ -12,7 +12,7 @@ import torch
 
 from ..kernels import elementwise as K
 from ..weights.loader import WeightSpec, WeightStore
-from .base import Block, FeedForward, KVNeed, LayerCache, Mixer, Norm, StateNeed, StepContext
+from .base import Block, FeedForward, KVNeed, LayerCache, Mixer, Norm, OpenSum, StateNeed, StepContext
 
 
 class PreNormBlock(Block):
@@ -204,6 +204,86 @@ class SandwichBlock(Block):
             xn = part.apply(x, ctx, cast=h if k == 0 else None, then=out_norm if k == n_after - 1 else None)
         if xn is not None and out_norm is not None:
             ctx.carry[NORMED_STREAM] = xn
+        return x, None
+
+
+class ParallelBlock(Block):
+    """One norm, both sub-layers on its output, one sum:
+
+        h = norm(x);  x += s1 * mixer(h) + s2 * feed_forward(h)
+
+    with a factor per element on each sub-layer's result (`mixer_scale`, `ffn_scale`: tensors of the width; None: no
+    factor).  The feed-forward may be absent.  Neither sub-layer waits for the other: the feed-forward runs on a second
+    stream beside the mixer, and the two meet in the sum.  leave_open: the sum is left to the norm that reads the stream
+    next (an OpenSum; a routed feed-forward's weighted sum over its experts joins it), which must be of a kind that
+    takes one; else the block adds it up itself."""
+
+    _side_streams = {}
+
+    def __init__(self, norm: Norm, mixer: Mixer, ffn: Optional[FeedForward] = None, hidden: int = 0,
+                 mixer_scale: Optional[str] = None, ffn_scale: Optional[str] = None, leave_open: bool = False):
+        if hidden < 1 or (ffn is None and ffn_scale is not None):
+            raise ValueError(f"block: width {hidden}; a feed-forward's factor comes with a feed-forward")
+        self.norm, self.mixer, self.ffn, self.hidden = norm, mixer, ffn, int(hidden)
+        self.scale_names, self.leave_open = (mixer_scale, ffn_scale), bool(leave_open)
+        self.scales: List[Optional[torch.Tensor]] = [None, None]
+
+    def parts(self):
+        return [p for p in (self.norm, self.mixer, self.ffn) if p is not None]
+
+    def cache_need(self) -> Optional[KVNeed]:
+        return self.mixer.cache_need()
+
+    def state_need(self) -> Optional[StateNeed]:
+        return self.mixer.state_need()
+
+    def capturable(self) -> bool:
+        return self.mixer.capturable() and (self.ffn is None or self.ffn.capturable())
+
+    def weight_specs(self) -> List[WeightSpec]:
+        return [s for p in self.parts() for s in p.weight_specs()] + \
+               [WeightSpec(n, (self.hidden,), init="one_plus_normal") for n in self.scale_names if n is not None]
+
+    def bind(self, store: WeightStore) -> None:
+        for p in self.parts():
+            p.bind(store)
+        self.scales = [None if n is None else store.get(n).float().contiguous() for n in self.scale_names]
+
+    def kernels(self) -> List[str]:
+        return ["elementwise"] + [k for p in self.parts() for k in p.kernels()]
+
+    @classmethod
+    def _side_stream(cls, device):
+        key = torch.device(device).index
+        if key not in cls._side_streams:
+            cls._side_streams[key] = torch.cuda.Stream(device=device)
+        return cls._side_streams[key]
+
+    def forward(self, x: torch.Tensor, pending, ctx: StepContext, cache: LayerCache):
+        if isinstance(pending, OpenSum) and not self.norm.adds_open_sums:
+            K.branches_dyt(x, **pending.operands())
+            pending = None
+        if pending is None:
+            h = self.norm.forward(x, ctx.act_dtype)
+        else:
+            h = self.norm.add_forward(x, pending, ctx.act_dtype)
+        f = None
+        if self.ffn is not None:
+            # what the feed-forward allocates on the second stream is read by the sum on this one and not used again
+            # before the second stream has waited for this one, at the next layer's fork: no block of memory is
+            # handed out while the other stream still reads it
+            main, side = torch.cuda.current_stream(), self._side_stream(x.device)
+            side.wait_stream(main)
+            with torch.cuda.stream(side):
+                f = self.ffn.forward(h, ctx, leave_rows=True) if hasattr(self.ffn, "n_experts") else self.ffn.forward(h, ctx)
+            y = self.mixer.forward(h, ctx, cache)
+            main.wait_stream(side)
+        else:
+            y = self.mixer.forward(h, ctx, cache)
+        both = OpenSum(y, self.scales[0], f, self.scales[1])
+        if self.leave_open:
+            return x, both
+        K.branches_dyt(x, **both.operands())
         return x, None
 
 

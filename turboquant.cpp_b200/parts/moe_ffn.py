@@ -14,7 +14,10 @@ Options other designs use: the experts' gated activation as constants (`glu`, `s
 a correction added to the scores for the choice only (`correction`: a tensor of one number per expert); groups of
 neighbouring experts of which only the `keep_groups` best (by their best corrected score) can be chosen; a floor
 added to the chosen scores' sum before the division (`renorm_floor`); a bias on the experts' logits (`router_bias`:
-a tensor of one number per expert, added before the choice and the weights); the tensors' names (`names`).
+a tensor of one number per expert, added before the choice and the weights); each logit's sigmoid as its score instead
+of the softmax over all (`scores`); a group's value as the sum of its two largest corrected scores (`group_top`);
+experts of two products with a function of one element between them instead of the gated three (`gated` False, `map`:
+W_down map(W_up x)); the tensors' names (`names`).
 """
 from __future__ import annotations
 
@@ -28,7 +31,7 @@ from ..kernels import gemm_tc as KT
 from ..kernels import moe as KM
 from ..kernels.linear import linear
 from ..weights.loader import WeightSpec, WeightStore
-from .base import FeedForward, StepContext, register_feed_forward
+from .base import ExpertRows, FeedForward, StepContext, register_feed_forward
 
 
 def KA_resident(device) -> int:
@@ -92,7 +95,14 @@ class MoEFeedForward(FeedForward):
                  norm_topk: bool, shared_intermediate: int = 0, shared_gate: bool = True,
                  glu: KE.Glu = KE.SILU_GLU, shared_glu: Optional[KE.Glu] = None, correction: bool = False,
                  n_groups: int = 1, keep_groups: int = 1, renorm_floor: float = 0.0, names=None,
-                 router_bias: bool = False):
+                 router_bias: bool = False, scores: str = "softmax", group_top: int = 1, gated: bool = True,
+                 map: int = KE.MAP_RELU_SQUARED):
+        """gated False: experts (and the shared one) have no gate, the function `map` (kernels.elementwise.MAP_*) stands
+        between their two products, and `glu` is not used."""
+        if scores not in ("softmax", "sigmoid") or group_top not in (1, 2):
+            raise ValueError(f"experts '{prefix}': scores '{scores}' (softmax or sigmoid), a group's value from its "
+                             f"{group_top} largest scores (1 or 2)")
+        self.sigmoid, self.group_top, self.gated, self.map = scores == "sigmoid", int(group_top), bool(gated), int(map)
         if n_experts < 1 or not 1 <= top_k <= n_experts:
             raise ValueError(f"experts '{prefix}': top-k {top_k} must be in 1..{n_experts}")
         if n_groups < 1 or n_experts % n_groups or not 1 <= keep_groups <= n_groups \
@@ -107,7 +117,7 @@ class MoEFeedForward(FeedForward):
         self.has_correction, self.n_groups, self.keep_groups = bool(correction), int(n_groups), int(keep_groups)
         self.renorm_floor = float(renorm_floor)
         # the choice needs more than the k largest logits: the selection kernel that knows corrections and groups
-        self.corrected = self.has_correction or self.n_groups > 1 or self.renorm_floor > 0.0
+        self.corrected = self.has_correction or self.n_groups > 1 or self.renorm_floor > 0.0 or self.sigmoid
         self.names = dict(QWEN_NAMES, **(names or {}))
         self.w_correction = None
         if hidden < 1 or intermediate < 1 or shared_intermediate < 0:
@@ -117,8 +127,12 @@ class MoEFeedForward(FeedForward):
         self.norm_topk, self.shared_intermediate = bool(norm_topk), int(shared_intermediate)
         self.shared_gate = bool(shared_gate) and shared_intermediate > 0
         self.w_router = self.w_shared_gate = self.w_router_packed = None
-        self.w13 = self.w2 = None            # [E, 2I, H] (gate rows, up rows), [E, H, I]
-        self.ws13 = self.ws2 = None          # shared expert [1, 2S, H], [1, H, S]
+        self.w13 = self.w2 = None            # [E, 2I, H] (gate rows, up rows; ungated: [E, I, H]), [E, H, I]
+        self.ws13 = self.ws2 = None          # shared expert [1, 2S, H] (ungated: [1, S, H]), [1, H, S]
+
+    def _inner(self):
+        """The products ahead of an expert's activation, in the order of their rows in the stacked weights."""
+        return ("gate", "up") if self.gated else ("up",)
 
     def weight_specs(self) -> List[WeightSpec]:
         p, H, I, S, n = self.prefix, self.hidden, self.intermediate, self.shared_intermediate, self.names
@@ -129,10 +143,10 @@ class MoEFeedForward(FeedForward):
             specs.append(WeightSpec(p + n["router_bias"], (self.n_experts,)))
         for e in range(self.n_experts):
             q = p + n["expert"].format(e=e)
-            specs += [WeightSpec(q + n["gate"], (I, H)), WeightSpec(q + n["up"], (I, H)), WeightSpec(q + n["down"], (H, I))]
+            specs += [WeightSpec(q + n[m], (I, H)) for m in self._inner()] + [WeightSpec(q + n["down"], (H, I))]
         if S > 0:
             q = p + n["shared"]
-            specs += [WeightSpec(q + n["gate"], (S, H)), WeightSpec(q + n["up"], (S, H)), WeightSpec(q + n["down"], (H, S))]
+            specs += [WeightSpec(q + n[m], (S, H)) for m in self._inner()] + [WeightSpec(q + n["down"], (H, S))]
             if self.shared_gate:
                 specs.append(WeightSpec(p + n["shared_gate"], (1, H)))
         return specs
@@ -147,20 +161,21 @@ class MoEFeedForward(FeedForward):
             self.w_router_bias = store.get(p + nm["router_bias"]).float().contiguous()
         # a tensor stored in 32 bits stays 32-bit: if any of the experts' tensors is kept in float32, the stacked
         # buffers are float32 (the others widen exactly), never the other way round
-        names = [p + nm["expert"].format(e=e) + nm[n] for e in range(E) for n in ("gate", "up", "down")]
+        names = [p + nm["expert"].format(e=e) + nm[n] for e in range(E) for n in self._inner() + ("down",)]
         dt = torch.float32 if any(store.kept_dtype_of(n) == torch.float32 for n in names) else store.kept_dtype_of(names[0])
-        self.w13 = torch.empty((E, 2 * I, H), dtype=dt, device=store.device)
+        inner = self._inner()
+        self.w13 = torch.empty((E, len(inner) * I, H), dtype=dt, device=store.device)
         self.w2 = torch.empty((E, H, I), dtype=dt, device=store.device)
         for e in range(E):
             q = p + nm["expert"].format(e=e)
-            self.w13[e, :I].copy_(store.take(q + nm["gate"]))
-            self.w13[e, I:].copy_(store.take(q + nm["up"]))
+            for j, m in enumerate(inner):
+                self.w13[e, j * I:(j + 1) * I].copy_(store.take(q + nm[m]))
             self.w2[e].copy_(store.take(q + nm["down"]))
         if S > 0:
             q = p + nm["shared"]
-            g, u, d = (store.take(q + nm[n]) for n in ("gate", "up", "down"))
-            sdt = torch.float32 if torch.float32 in (g.dtype, u.dtype, d.dtype) else g.dtype
-            self.ws13 = torch.cat([g.to(sdt), u.to(sdt)], dim=0).unsqueeze(0).contiguous()
+            *up, d = (store.take(q + nm[n]) for n in inner + ("down",))
+            sdt = torch.float32 if torch.float32 in [t.dtype for t in up] + [d.dtype] else d.dtype
+            self.ws13 = torch.cat([t.to(sdt) for t in up], dim=0).unsqueeze(0).contiguous()
             self.ws2 = d.to(sdt).unsqueeze(0).contiguous()
             if self.shared_gate:
                 self.w_shared_gate = store.get(p + nm["shared_gate"])
@@ -174,11 +189,11 @@ class MoEFeedForward(FeedForward):
         # bfloat16 runs whose sizes give 16-byte rows keep the expert weights only in the packed layout
         # of the tensor-core kernel
         if store.run_dtype == torch.bfloat16 and H % 8 == 0 and I % 8 == 0 and KT.packable(self.w13) and KT.packable(self.w2):
-            self.w13 = KT.pack_weights(self.w13, True)
+            self.w13 = KT.pack_weights(self.w13, self.gated)
             self.w2 = KT.pack_weights(self.w2, False)
         if self.ws13 is not None and store.run_dtype == torch.bfloat16 and H % 8 == 0 and S % 8 == 0 \
                 and KT.packable(self.ws13) and KT.packable(self.ws2):
-            self.ws13 = KT.pack_weights(self.ws13, True)
+            self.ws13 = KT.pack_weights(self.ws13, self.gated)
             self.ws2 = KT.pack_weights(self.ws2, False)
 
     def kernels(self) -> List[str]:
@@ -191,9 +206,9 @@ class MoEFeedForward(FeedForward):
     def step_work(self, n_tokens, kv_tokens):
         E, k, H, I, S = self.n_experts, self.top_k, self.hidden, self.intermediate, self.shared_intermediate
         el = 4 if getattr(self, "run_dtype", None) == torch.float32 else 2
-        touched = experts_touched(n_tokens, E, k)
-        byt = el * (touched * 3 * H * I + 3 * H * S + (E + 1) * H)
-        return {"moe": (byt, 2.0 * n_tokens * (k * 3 * H * I + 3 * H * S + (E + 1) * H))}
+        touched, m = experts_touched(n_tokens, E, k), len(self._inner()) + 1
+        byt = el * (touched * m * H * I + m * H * S + (E + 1) * H)
+        return {"moe": (byt, 2.0 * n_tokens * (k * m * H * I + m * H * S + (E + 1) * H))}
 
     _side_streams = {}
 
@@ -208,17 +223,18 @@ class MoEFeedForward(FeedForward):
     EXACT_SHARED_ROWS = 2        # rows of the shared expert that the exact weight-stream kernel takes in one pass
     EXACT_FEW_ROWS = int(os.environ.get("TQ_EXACT_FEW_ROWS", "64"))      # steps of up to this many tokens take the exact kernels' weight-stream form
 
-    def _product(self, x, w, out, layout, swiglu, token_tile, status=None, early=False, glu=None):
+    def _product(self, x, w, out, layout, inner, token_tile, status=None, early=False, glu=None):
         """Tensor cores for weights packed at load time (bfloat16, 16-byte rows), the exact CUDA-core
-        kernel otherwise.  early: this is a down projection right behind its gate/up product in the stream: its
+        kernel otherwise.  inner: the product(s) ahead of the activation, which rides on it.  early: this is a down projection right behind its gate/up product in the stream: its
         weights and the layout were there before that product started, so it may stream weights while that runs."""
+        swiglu, map = inner and self.gated, self.map if inner and not self.gated else KE.MAP_COPY
         if isinstance(w, KT.PackedWeights):
-            return KT.gemm_tc(x, w, out, layout, token_tile, status=status, early_weights=early and self.EARLY_WEIGHTS, glu=glu)
+            return KT.gemm_tc(x, w, out, layout, token_tile, status=status, early_weights=early and self.EARLY_WEIGHTS, glu=glu, map=map)
         # the exact kernels: tiles of a few rows (decode steps) stream the weights; a group's tile holds at most the
         # step's tokens, and the one-group product (the shared expert) all of them
         rows = x.shape[0]
         few = rows <= self.EXACT_FEW_ROWS if layout is None else rows <= self.EXACT_FEW_ROWS * self.top_k
-        return KM.grouped_gemm(x, w, out, layout, swiglu, few_rows=few, glu=glu)
+        return KM.grouped_gemm(x, w, out, layout, swiglu, few_rows=few, glu=glu, map=map)
 
     def _joint_launches(self, T: int, tile: int, act, dev) -> bool:
         """Whether the shared expert's two products ride in the routed experts' launches, their tiles ahead of the
@@ -232,14 +248,16 @@ class MoEFeedForward(FeedForward):
         either: both draw on the L2's bandwidth.  Giving each product a share of the SMs instead, as launches of
         their own on two streams, cost 25-60 %.)"""
         how = self.SHARED_IN_ROUTED_LAUNCH
-        if (self.ws13 is None or tile < KT.PAIR_MIN_TILE or KT._NO_PAIRS or how == "0" or act != torch.bfloat16
+        if (self.ws13 is None or not self.gated or tile < KT.PAIR_MIN_TILE or KT._NO_PAIRS or how == "0" or act != torch.bfloat16
                 or not all(isinstance(w, KT.PackedWeights) for w in (self.w13, self.w2, self.ws13, self.ws2))):
             return False
         if how != "":
             return True
         return shared_rides_with_routed(T, self.shared_intermediate, KA_resident(dev))
 
-    def forward(self, xn: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+    def forward(self, xn: torch.Tensor, ctx: StepContext, leave_rows: bool = False):
+        """leave_rows: the last step, the weighted sum of each token's rows, is left to the caller where nothing else
+        is in it (no shared expert): ExpertRows instead of the sum."""
         T, H, k, dev = xn.shape[0], self.hidden, self.top_k, xn.device
         act = ctx.act_dtype
         # the shared expert does not depend on the routing: it runs on a second stream next to the routed experts
@@ -264,6 +282,10 @@ class MoEFeedForward(FeedForward):
         # A2.7B sizes batch 8: 2,214 / 2,287, batch 16: 3,228 / 3,147; 57B-A14B sizes batch 1: 177 / 190, batch 8: 602 / 586.)
         shared_after = small and (T * k >= self.n_experts if self.SHARED_AFTER_ROUTER is None else self.SHARED_AFTER_ROUTER)
 
+        def select(logits):
+            KM.router_select_corrected(logits, self.w_correction, k, self.norm_topk, self.renorm_floor, self.n_groups,
+                                       self.keep_groups, ids, wts, scale, sigmoid=self.sigmoid, group_top=self.group_top)
+
         def shared_expert():
             nonlocal y_shared, side
             S = self.shared_intermediate
@@ -278,7 +300,10 @@ class MoEFeedForward(FeedForward):
                     # one pass of the exact weight-stream kernel holds: the shared expert is a dense feed-forward, and
                     # the library's products serve it as they serve the dense layers
                     gu = linear(xn, self.ws13[0], out_dtype=torch.float32)
-                    KE.glu_mul(gu, hs, self.shared_glu)
+                    if self.gated:
+                        KE.glu_mul(gu, hs, self.shared_glu)
+                    else:
+                        KE.map_elements(gu, hs, self.map)
                     y_shared = linear(hs, self.ws2[0], out_dtype=torch.float32)
                     return
                 self._product(xn, self.ws13, hs, None, True, stile, ctx.status, glu=self.shared_glu)
@@ -301,7 +326,8 @@ class MoEFeedForward(FeedForward):
             # few tokens (decoding): router, layout and the sorted copies of the rows in one launch
             KM.router_small(xn, self.w_router, self.w_shared_gate, k, self.norm_topk, ids, wts, scale, layout, x_rows,
                             correction=self.w_correction, corrected=self.corrected, floor=self.renorm_floor,
-                            n_groups=self.n_groups, keep_groups=self.keep_groups, logit_bias=self.w_router_bias)
+                            n_groups=self.n_groups, keep_groups=self.keep_groups, logit_bias=self.w_router_bias,
+                            sigmoid=self.sigmoid, group_top=self.group_top)
         else:
             if self.w_router_packed is not None and T >= self.ROUTER_TC_MIN_TOKENS:
                 # long steps (prompts): the logits of all tokens as one tensor-core product (bf16 x bf16 products
@@ -311,16 +337,14 @@ class MoEFeedForward(FeedForward):
                 if self.w_router_bias is not None:
                     KE.scale_bias_cols(logits, 1.0, self.w_router_bias, cols=self.n_experts)
                 if self.corrected:
-                    KM.router_select_corrected(logits, self.w_correction, k, self.norm_topk, self.renorm_floor,
-                                               self.n_groups, self.keep_groups, ids, wts, scale)
+                    select(logits)
                 else:
                     KM.router_select(logits, k, self.norm_topk, ids, wts, scale)
             elif self.corrected:
                 logits = KM.router_logits(xn, self.w_router, self.w_shared_gate,
                                           torch.empty((T, self.n_experts + 1), dtype=torch.float32, device=dev),
                                           logit_bias=self.w_router_bias)
-                KM.router_select_corrected(logits, self.w_correction, k, self.norm_topk, self.renorm_floor,
-                                           self.n_groups, self.keep_groups, ids, wts, scale)
+                select(logits)
             else:
                 KM.router_topk(xn, self.w_router, self.w_shared_gate, k, self.norm_topk, ids, wts, scale,
                                logit_bias=self.w_router_bias)
@@ -347,6 +371,8 @@ class MoEFeedForward(FeedForward):
             self._product(h_rows, self.w2, y_rows, layout, False, tile, ctx.status, early=True)
         if side is not None:
             torch.cuda.current_stream().wait_stream(side)
+        if leave_rows and y_shared is None:
+            return ExpertRows(y_rows, layout.row_of_pair, wts)
         y = torch.empty((T, H), dtype=torch.float32, device=dev)
         KM.moe_combine(y_rows, layout.row_of_pair, wts, y_shared, scale, y, k)
         return y

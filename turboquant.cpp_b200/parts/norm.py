@@ -8,7 +8,7 @@ import torch
 
 from ..kernels import elementwise as K
 from ..weights.loader import WeightSpec, WeightStore
-from .base import Norm, register_norm
+from .base import Norm, OpenSum, register_norm
 
 
 class RMSNorm(Norm):
@@ -74,7 +74,10 @@ class DynamicTanh(Norm):
     """A norm without statistics: y = tanh(alpha * x) * w + b, with a learned scalar alpha (tensor `<name>.alpha`), a
     weight `<name>` and a bias `<name>.b`.  Reads the fp32 residual stream; computed in fp32.  The sums that other
     norms take along (`add`, `add_forward`) may carry a factor: x += scale * y.  `shifted()` mixes every token's
-    output with that of the token before it (see there)."""
+    output with that of the token before it (see there).  They may also be an OpenSum, two sub-layers' outputs with a
+    factor per element."""
+
+    adds_open_sums = True
 
     def __init__(self, name: str, size: int):
         if size < 1:
@@ -100,10 +103,19 @@ class DynamicTanh(Norm):
     def forward(self, x, out_dtype, rows=None, add=None, add_scale: float = 1.0):
         n = x.shape[0] if rows is None else rows.shape[0]
         out = torch.empty((n, self.size), dtype=out_dtype, device=x.device)
+        if isinstance(add, OpenSum):
+            return self._of_open_sum(x, add, add_scale, out, rows)
         return K.dyt(x, self.alpha, self.weight, self.bias, out, add=add, add_scale=add_scale, rows=rows)
+
+    def _of_open_sum(self, x, add, scale, out, rows=None):
+        if scale != 1.0:
+            raise ValueError(f"DynamicTanh '{self.name}': an open sum carries its factors itself")
+        return K.branches_dyt(x, rows=rows, alpha=self.alpha, weight=self.weight, bias=self.bias, out=out, **add.operands())
 
     def add_forward(self, x, y, out_dtype, scale: float = 1.0):
         out = torch.empty((x.shape[0], self.size), dtype=out_dtype, device=x.device)
+        if isinstance(y, OpenSum):
+            return self._of_open_sum(x, y, scale, out)
         return K.dyt(x, self.alpha, self.weight, self.bias, out, add=y, add_scale=scale)
 
     def shifted(self, x, out_dtype, shift: torch.Tensor, kept: torch.Tensor, ctx) -> torch.Tensor:
