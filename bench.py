@@ -150,7 +150,7 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 / 64 points and the prefill")
     ap.add_argument("--kernel-table", default="", help="write a per-kernel time table of a few decode steps and of a "
                     "prefill to this file (torch profiler; not part of any timed number)")
-    ap.add_argument("--design", choices=["nuforax", "lumevik", "sisepel", "tasadra"], default="", help="instead of the default workload: prompt "
+    ap.add_argument("--design", choices=["nuforax", "lumevik", "sisepel", "tasadra", "vukotar"], default="", help="instead of the default workload: prompt "
                     "and decode speed of this design at layer sizes of a real model (random weights), beside the closest other "
                     "decoder of equal width, depth and heads")
     ap.add_argument("--sizes", default="w1024,w2048", help="with --design: which of the sizes to run")
@@ -483,6 +483,8 @@ def design_compare(args) -> int:
         return sisepel_compare(args, tq, measure, weights_bytes, pk, rng, prompt, steps, warmup)
     if args.design == "tasadra":
         return tasadra_compare(args, tq, measure, weights_bytes, pk, rng, prompt, steps, warmup)
+    if args.design == "vukotar":
+        return vukotar_compare(args, tq, measure, pk, rng, prompt, steps, warmup)
     result = {"metric": "prompt and decode speed, Nuforax beside the dense Qwen2 decoder of equal width", "unit": "tokens/s",
               "n_gpus": 1, "steps": steps, "warmup": warmup, "dtype": "bf16", "data": "synthetic token ids, seeded random weights",
               "peaks": pk, "sizes": {}}
@@ -659,8 +661,89 @@ def tasadra_compare(args, tq, measure, weights_bytes, pk, rng, prompt, steps, wa
     return 0
 
 
-def kernel_table(tq, model, rng, V, batch, path, prompt=None, context=None):
-    """Per-kernel device time of 4 decode steps at context 2,048 and of one 2,048-token prefill."""
+def vukotar_config(width, layers, heads, kv_heads, dim, experts, top, e_ff, vocab):
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5}
+    moe = {"kind": "moe", "expert": {"ff": e_ff}, "router": {"experts": experts, "top": top, "groups": {"count": 4, "keep": 2}}}
+    return {"architecture": "Vukotar", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": width ** 0.5},
+            "logit_softcap": 50.0, "layers": [{"type": "attention", "mixer": att, "mlp": moe}] * layers}
+
+
+def lumevik_routed_config(width, layers, heads, kv_heads, dim, experts, top, e_ff, vocab):
+    """The Lumevik decoder with attention over every earlier position and routed experts on every layer, without shared
+    expert and value mixing."""
+    att = {"type": "attention", "mlp": {"kind": "moe", "expert": {"ff": e_ff, "limit": 7.0},
+                                        "router": {"experts": experts, "top": top, "groups": {"count": 4, "keep": 2}}},
+           "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "bias_max": 2048, "bias_rows": 32}}
+    return {"architecture": "Lumevik", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": [att] * layers}
+
+
+VUKOTAR_SIZES = {
+    # name: (width, layers, heads, kv heads, head size, experts, top, ff of an expert of two products, of one of three, vocab)
+    "w1024": (1024, 4, 8, 2, 128, 32, 4, 1056, 704, 32768),
+    "w2048": (2048, 4, 16, 4, 128, 60, 4, 2112, 1408, 32768),
+}
+
+
+def experts_chosen(tq, model, rng, V, batch):
+    """Distinct experts per routed layer that one decode step of `batch` sequences reads (short random contexts)."""
+    import torch
+    eng = tq.Engine(model, max_tokens=batch * 64, max_slots=batch)
+    seqs = [eng.open() for _ in range(batch)]
+    eng.step([tq.StepEntry(s, rng.integers(0, V, size=16).tolist(), []) for s in seqs])
+    eng.debug = {}
+    eng.step([tq.StepEntry(s, [int(rng.integers(0, V))], [0]) for s in seqs])
+    n = [int(torch.unique(ids).numel()) for ids in eng.debug["router_ids"]]
+    for s in seqs:
+        eng.close(s)
+    eng.release()
+    return n
+
+
+def vukotar_compare(args, tq, measure, pk, rng, prompt, steps, warmup) -> int:
+    """The Vukotar decoder beside the Lumevik decoder of the same width, depth, heads, experts and weights per expert: both
+    run attention with one more in the denominator on the same kernels and grouped routing; Lumevik adds a distance
+    bias and a gate in its experts (whose inner size is smaller for that), and runs its sub-layers one after the other."""
+    import torch
+    result = {"metric": "prompt and decode speed, Vukotar beside the Lumevik decoder of equal sizes", "unit": "tokens/s",
+              "n_gpus": 1, "steps": steps, "warmup": warmup, "dtype": "bf16", "data": "synthetic token ids, seeded random weights",
+              "peaks": pk, "sizes": {}}
+    clocks = ClockSampler()
+    clocks.start()
+    for name in args.sizes.split(","):
+        if name not in VUKOTAR_SIZES:
+            print(json.dumps({"error": f"unknown size '{name}'; known: {sorted(VUKOTAR_SIZES)}"}))
+            return 2
+        (W, L, H, G, D, E, top, ff2, ff3, V) = VUKOTAR_SIZES[name]
+        entry = {}
+        for who, cfg, ff in (("vukotar", vukotar_config(W, L, H, G, D, E, top, ff2, V), ff2),
+                             ("lumevik", lumevik_routed_config(W, L, H, G, D, E, top, ff3, V), ff3)):
+            model = tq.random_model(cfg, seed=0, dtype="bfloat16", device="cuda:0")
+            entry[who] = dict(measure(model, V), config={"width": W, "layers": L, "heads": H, "kv_heads": G, "head_size": D,
+                                                         "experts": E, "top": top, "expert_ff": ff})
+            for batch in (1, 8, 64):
+                # the bytes a decode step reads: everything but the experts once, the experts its tokens chose, the live rows
+                n = experts_chosen(tq, model, rng, V, batch)
+                per = (2 if who == "vukotar" else 3) * W * ff * 2
+                d = entry[who][f"decode_b{batch}"]
+                read = L * (2 * W * (H + G) * D + E * W) * 2 + V * W * 2 + sum(n) * per + L * batch * prompt * 2 * G * D * 2
+                d.update(experts_per_layer=round(sum(n) / L, 1), read_gb=round(read / 1e9, 4),
+                         frac_of_copy_peak=round(read / (d["ms_per_step"] * 1e-3) / 1e9 / pk["hbm_gbs"], 4))
+                d.pop("weights_frac_of_copy_peak")
+            if args.kernel_table:
+                kernel_table(tq, model, rng, V, args.batch, args.kernel_table + f".{who}_{name}.txt", prompt=prompt,
+                             context=prompt + 128, same_token=False)
+            del model
+            gc.collect()
+            torch.cuda.empty_cache()
+        result["sizes"][name] = entry
+    result["clocks"] = clocks.stop()
+    print(json.dumps(result))
+    return 0
+
+
+def kernel_table(tq, model, rng, V, batch, path, prompt=None, context=None, same_token=True):
+    """Per-kernel device time of 4 decode steps at context 2,048 and of one 2,048-token prefill.  same_token: every sequence
+    of the decode steps brings token 1 (else tokens at random, which spreads a step over more experts)."""
     import torch
     from torch.profiler import ProfilerActivity, profile
     PROMPT, CONTEXT = prompt or globals()["PROMPT"], context or globals()["CONTEXT"]
@@ -668,7 +751,7 @@ def kernel_table(tq, model, rng, V, batch, path, prompt=None, context=None):
     seqs = [eng.open() for _ in range(batch)]
     for g0 in range(0, batch, 8):
         eng.step([tq.StepEntry(s, rng.integers(0, V, size=PROMPT).tolist(), []) for s in seqs[g0:g0 + 8]])
-    step = lambda: eng.step([tq.StepEntry(s, [1], [0]) for s in seqs])
+    step = lambda: eng.step([tq.StepEntry(s, [1 if same_token else int(rng.integers(0, V))], [0]) for s in seqs])
     step()
     torch.cuda.synchronize()
     with profile(activities=[ProfilerActivity.CUDA]) as prof:

@@ -13,8 +13,24 @@ from vukotar_util import CONFIGS, attention, config, layer, make_weights, moe, t
 def test_the_models_plan_names_every_tensor_with_its_shape():
     import turboquant_cpp_b200 as tq
     for name, cfg in CONFIGS.items():
-        plan = {s.name: tuple(s.shape) for s in tq.build_model(cfg, "bfloat16").weight_specs()}
-        assert plan == tensor_shapes(cfg), name
+        specs = tq.build_model(cfg, "bfloat16").weight_specs()
+        assert {s.name: tuple(s.shape) for s in specs if not s.optional} == tensor_shapes(cfg), name
+        # the factor of a feed-forward that a layer does not have may be stored or not
+        assert [s.name for s in specs if s.optional] == (["l1.ls2"] if name == "a" else [])
+
+
+def test_a_tensor_nothing_reads_may_be_left_out_and_any_other_may_not():
+    import torch
+    import turboquant_cpp_b200 as tq
+    from turboquant_cpp_b200.weights import WeightError, check_plan
+    specs = tq.build_model(CONFIGS["a"], "bfloat16").weight_specs()
+    index = {n: (torch.bfloat16, s) for n, s in tensor_shapes(CONFIGS["a"]).items()}
+    check_plan(index, specs)
+    check_plan(dict(index, **{"l1.ls2": (torch.bfloat16, (CONFIGS["a"]["width"],))}), specs)
+    with pytest.raises(WeightError, match="l1.ls2"):
+        check_plan(dict(index, **{"l1.ls2": (torch.bfloat16, (3,))}), specs)
+    with pytest.raises(WeightError, match="l0.ls2"):
+        check_plan({n: v for n, v in index.items() if n != "l0.ls2"}, specs)
 
 
 def test_layers_that_share_weights_run_one_block_with_caches_of_their_own():

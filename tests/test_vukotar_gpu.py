@@ -213,7 +213,7 @@ def test_a_far_token_reaches_through_every_page(tmp_path):
     engine follows that change in a prompt, in decoding and across portions."""
     cfg = config([layer(attention(heads=2, kv_heads=1, dim=16, vdim=16, scale=1.0), moe(experts=4, top=1, groups=(2, 1), ff=16)),
                   layer(attention(heads=2, kv_heads=1, dim=16, vdim=16, scale=1.0), moe(experts=4, top=1, groups=(2, 1), ff=16), weights_of=0)],
-                 vocab=40, width=32, scale=3.0, cap=30.0)
+                 vocab=40, width=32, scale=3.0, cap=25.0)
     w = make_weights(cfg, 9)
     w["l0.mix.q"] = w["l0.mix.q"] * 0.05                                  # flat weights: every far token counts a little
     folder = write_folder(str(tmp_path / "far"), cfg, w)
@@ -294,3 +294,84 @@ def test_command_line_and_trace_replay(folders, tmp_path):
     ref = plain_model(folder).forward(toks)
     got = np.concatenate([np.fromfile(tmp_path / "o" / f"{s}.f32", dtype="<f4").reshape(-1, cfg["vocab"]) for s in (0, 2)])
     assert np.abs(got - ref[[0, 29, 39]]).max() < 1e-4 * ref.std()
+
+
+@pytest.mark.parametrize("T", [1, 6, 40, 700])
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_ungated_experts_beside_a_shared_one(T, dtype):
+    """The routed part with an option this design leaves out: a shared expert without a gate inside it (beside the routed
+    experts on a second stream, its output weighted by a gate of its own)."""
+    import types
+    import torch
+    from plain import vukotar_plain as P
+    from turboquant_cpp_b200.parts import ExpertRows, make_feed_forward
+    from turboquant_cpp_b200.weights import RandomSource, WeightStore
+    H, E, k, I, S = 64, 10, 3, 24, 72
+    names = {"router": "router", "expert": "e{e}.", "up": "up", "down": "down", "shared": "sh.", "shared_gate": "sg"}
+    run = torch.float32 if dtype == "float32" else torch.bfloat16
+    for shared in (S, 0):
+        ff = make_feed_forward("moe", prefix="f.", hidden=H, n_experts=E, top_k=k, intermediate=I, norm_topk=True,
+                               shared_intermediate=shared, n_groups=5, keep_groups=3, group_top=2, scores="sigmoid",
+                               renorm_floor=P.WEIGHT_FLOOR, gated=False, names=names)
+        specs = ff.weight_specs()
+        store = WeightStore(RandomSource(specs, 4, std=0.2), specs, "cuda:0", run)
+        w = {s.name: store.get(s.name).double().cpu().numpy() for s in specs}
+        assert not any("gate" in n for n in w)
+        ff.bind(store)
+        x = torch.randn(T, H, device="cuda:0").to(run)
+        ctx = types.SimpleNamespace(act_dtype=run, debug={}, status=None)
+        y = ff.forward(x, ctx)
+        h, ids = x.double().cpu().numpy(), ctx.debug["router_ids"][0].cpu().numpy()
+        ml = {"router": {"experts": E, "top": k, "groups": {"count": 5, "keep": 3}}}
+        rec = []
+        P.experts(h, w, "f.", ml, record=rec)
+        differ = np.any(np.sort(ids, axis=1) != np.sort(rec[0][0], axis=1), axis=1)
+        assert rec[0][2][differ].max(initial=0.0) < 1e-5
+        want = P.experts(h, w, "f.", ml, ids=ids)
+        if shared:
+            want += P.expert(h, w, "f.sh.") / (1.0 + np.exp(-(h @ w["f.sg"].T)))
+        got = y.double().cpu().numpy()
+        assert np.abs(got - want).max() < (1e-5 if dtype == "float32" else 2e-2) * np.abs(want).max()
+        left = ff.forward(x, ctx, leave_rows=True)
+        assert isinstance(left, ExpertRows) == (shared == 0)
+
+
+def test_a_blocks_sum_left_open_or_not_and_the_two_streams_give_the_same(folders):
+    """The block with its sum taken by the next norm, with a sum of its own, with the feed-forward behind the mixer on one
+    stream, and with a norm that takes no open sum."""
+    import torch
+    import turboquant_cpp_b200 as tq
+    from turboquant_cpp_b200.parts import ParallelBlock
+    cfg, folder = CONFIGS["a"], folders["a"]
+    toks = tokens_for(cfg, 70, 5)
+
+    def logits(change, dtype="float32"):
+        model = tq.load_model(folder, dtype)
+        change(model)
+        eng = tq.Engine(model, max_tokens=128)
+        s = eng.open()
+        out = eng.step([tq.StepEntry(s, toks, list(range(70)))])
+        eng.close(s)
+        eng.release()
+        return out
+
+    ref = logits(lambda m: None)
+
+    def closed(m):
+        for b in m.blocks:
+            b.leave_open = False
+    assert (logits(closed) - ref).abs().max().item() < 1e-5 * ref.abs().max().item()
+
+    def other_norm(m):                                   # as if the norms that follow took sums of one tensor only
+        for b in m.blocks:
+            b.norm.adds_open_sums = False
+    assert (logits(other_norm) - ref).abs().max().item() < 1e-5 * ref.abs().max().item()
+    saved = ParallelBlock.SIDE_BY_SIDE, ParallelBlock.SIDE_MIN_ELEMENTS
+    try:
+        ParallelBlock.SIDE_MIN_ELEMENTS = 0                # two streams, whatever the step's size
+        for _ in range(3):
+            assert torch.equal(logits(lambda m: None), ref)
+        ParallelBlock.SIDE_BY_SIDE = False
+        assert torch.equal(logits(lambda m: None), ref)
+    finally:
+        ParallelBlock.SIDE_BY_SIDE, ParallelBlock.SIDE_MIN_ELEMENTS = saved

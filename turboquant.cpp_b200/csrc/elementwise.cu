@@ -1098,11 +1098,15 @@ TQ_EXPORT int tq_branches_dyt(float* x, const float* a, const float* s1, const f
 // x[t, j] = table[tokens[t], j] * scale + (j even: sin, odd: cos of 2 pi * positions[t] * turns[j / 2])
 // turns: a position's step in full turns per pair of columns, fp64 [(H + 1) / 2].  The turns are counted in fp64 and
 // only what is left of the last full one goes to fp32, so a far position's angle is as exact as a near one's.
+// wide: rows start on a pair's boundary (H even, aligned tensors), a pair is one access.
 // ---------------------------------------------------------------------------------------
+__device__ __forceinline__ float2 load_pair(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 load_pair(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+
 template <typename TW>
 __global__ void embed_position_rows_kernel(const int* __restrict__ tokens, const int* __restrict__ positions,
                                            const TW* __restrict__ table, const double* __restrict__ turns,
-                                           float* __restrict__ x, int H, int V, float scale) {
+                                           float* __restrict__ x, int H, int V, float scale, int wide) {
     tq_grid_wait();                    // everything below may read what the previous kernel wrote
     tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
     const int t = blockIdx.x;
@@ -1113,6 +1117,11 @@ __global__ void embed_position_rows_kernel(const int* __restrict__ tokens, const
         const double full = p * turns[m];
         float sn, cs;
         sincospif((float)(2.0 * (full - rint(full))), &sn, &cs);
+        if (wide) {
+            const float2 e = load_pair(row + 2 * m);
+            *reinterpret_cast<float2*>(out + 2 * m) = make_float2(e.x * scale + sn, e.y * scale + cs);
+            continue;
+        }
         out[2 * m] = tq_to_float(row[2 * m]) * scale + sn;
         if (2 * m + 1 < H) out[2 * m + 1] = tq_to_float(row[2 * m + 1]) * scale + cs;
     }
@@ -1122,10 +1131,11 @@ TQ_EXPORT int tq_embed_position_rows(const int* tokens, const int* positions, co
                                      float* x, int T_, int H, int V, float scale, cudaStream_t stream) {
     if (T_ == 0) return 0;
     TQ_REQUIRE(T_ > 0 && H > 0 && turns != nullptr, "embed_position_rows: bad sizes T=%d H=%d, or no table of turns", T_, H);
+    const int wide = H % 2 == 0 && ((uintptr_t)table & 7) == 0 && ((uintptr_t)x & 7) == 0;
     const int pairs = (H + 1) / 2, threads = pairs >= 512 ? 256 : 128;
     TQ_DISPATCH(table_dtype, TW,
         tq_launch(dim3(T_, (pairs + threads - 1) / threads), threads, 0, stream)(embed_position_rows_kernel<TW>, tokens, positions,
-            (const TW*)table, turns, x, H, V, scale));
+            (const TW*)table, turns, x, H, V, scale, wide));
     TQ_CHECK_LAUNCH("embed_position_rows");
     return 0;
 }

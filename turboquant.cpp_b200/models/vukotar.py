@@ -40,7 +40,7 @@ class VukotarModel(DecoderModel):
                                         gated=False, map=MAP_RELU_SQUARED, names=MOE_NAMES)
             block_of[i] = len(blocks)
             blocks.append(ParallelBlock(norm(p + "norm1"), mixer, ffn, hidden=W, mixer_scale=p + "ls1",
-                                        ffn_scale=p + "ls2" if ffn is not None else None, leave_open=True))
+                                        ffn_scale=p + "ls2", leave_open=True))
         schedule = [ScheduleEntry(block_of[i if layer.weights_of is None else layer.weights_of])
                     for i, layer in enumerate(cfg.layers)]
         super().__init__(cfg, dtype, embedding=PositionedEmbedding("embed", cfg.vocab, W, cfg.embedding_scale, POSITION_BASE),

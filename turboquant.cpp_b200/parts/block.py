@@ -6,6 +6,7 @@ sub-layer's output as `pending` and hands its own feed-forward output on the sam
 sum is one fp32 pass together with the next norm's statistics."""
 from __future__ import annotations
 
+import os
 from typing import List, Optional, Tuple
 
 import torch
@@ -219,11 +220,17 @@ class ParallelBlock(Block):
     takes one; else the block adds it up itself."""
 
     _side_streams = {}
+    SIDE_BY_SIDE = os.environ.get("TQ_NO_SIDE_BY_SIDE", "") in ("", "0")
+    # prompts whose stream holds fewer elements run on one stream: launches, not the GPU, bound such a step, and the fork
+    # and join are launches too (measured on B200, ms of a 2,048-token prompt through four layers on one stream / two:
+    # width 1,024: 1.60 / 1.68, width 2,048: 2.57 / 2.43); decode steps are replayed as graphs
+    SIDE_MIN_ELEMENTS = 3 << 20
 
     def __init__(self, norm: Norm, mixer: Mixer, ffn: Optional[FeedForward] = None, hidden: int = 0,
                  mixer_scale: Optional[str] = None, ffn_scale: Optional[str] = None, leave_open: bool = False):
-        if hidden < 1 or (ffn is None and ffn_scale is not None):
-            raise ValueError(f"block: width {hidden}; a feed-forward's factor comes with a feed-forward")
+        """ffn_scale without a feed-forward: the name of a tensor that a file may hold although nothing reads it."""
+        if hidden < 1:
+            raise ValueError(f"block: width {hidden}")
         self.norm, self.mixer, self.ffn, self.hidden = norm, mixer, ffn, int(hidden)
         self.scale_names, self.leave_open = (mixer_scale, ffn_scale), bool(leave_open)
         self.scales: List[Optional[torch.Tensor]] = [None, None]
@@ -242,12 +249,14 @@ class ParallelBlock(Block):
 
     def weight_specs(self) -> List[WeightSpec]:
         return [s for p in self.parts() for s in p.weight_specs()] + \
-               [WeightSpec(n, (self.hidden,), init="one_plus_normal") for n in self.scale_names if n is not None]
+               [WeightSpec(n, (self.hidden,), init="one_plus_normal", optional=part is None)
+                for n, part in zip(self.scale_names, (self.mixer, self.ffn)) if n is not None]
 
     def bind(self, store: WeightStore) -> None:
         for p in self.parts():
             p.bind(store)
-        self.scales = [None if n is None else store.get(n).float().contiguous() for n in self.scale_names]
+        self.scales = [None if n is None or part is None else store.get(n).float().contiguous()
+                       for n, part in zip(self.scale_names, (self.mixer, self.ffn))]
 
     def kernels(self) -> List[str]:
         return ["elementwise"] + [k for p in self.parts() for k in p.kernels()]
@@ -268,18 +277,20 @@ class ParallelBlock(Block):
         else:
             h = self.norm.add_forward(x, pending, ctx.act_dtype)
         f = None
-        if self.ffn is not None:
+        run_ffn = lambda: self.ffn.forward(h, ctx, leave_rows=True) if hasattr(self.ffn, "n_experts") else self.ffn.forward(h, ctx)
+        if self.ffn is not None and self.SIDE_BY_SIDE and (ctx.max_q_len == 1 or x.numel() >= self.SIDE_MIN_ELEMENTS):
             # what the feed-forward allocates on the second stream is read by the sum on this one and not used again
             # before the second stream has waited for this one, at the next layer's fork: no block of memory is
             # handed out while the other stream still reads it
             main, side = torch.cuda.current_stream(), self._side_stream(x.device)
             side.wait_stream(main)
             with torch.cuda.stream(side):
-                f = self.ffn.forward(h, ctx, leave_rows=True) if hasattr(self.ffn, "n_experts") else self.ffn.forward(h, ctx)
+                f = run_ffn()
             y = self.mixer.forward(h, ctx, cache)
             main.wait_stream(side)
         else:
             y = self.mixer.forward(h, ctx, cache)
+            f = run_ffn() if self.ffn is not None else None
         both = OpenSum(y, self.scales[0], f, self.scales[1])
         if self.leave_open:
             return x, both

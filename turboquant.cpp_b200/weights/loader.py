@@ -39,11 +39,13 @@ class WeightError(ValueError):
 
 @dataclass(frozen=True)
 class WeightSpec:
-    """shape: a dimension of -1 is read from the stored tensor (a table whose length no configuration key gives)."""
+    """shape: a dimension of -1 is read from the stored tensor (a table whose length no configuration key gives).
+    optional: a source may leave the tensor out (nothing in the model reads it)."""
     name: str
     shape: Tuple[int, ...]
     init: str = "normal"        # 'normal' | 'one_plus_normal' | 'zeros' | 'ones' | 'int_range'
     integer: bool = False        # an integer table (kept as int32)
+    optional: bool = False
 
 
 def run_dtype_of(name: str) -> torch.dtype:
@@ -108,7 +110,7 @@ def check_plan(index: Dict[str, Tuple[torch.dtype, Tuple[int, ...]]], plan: Sequ
         if s.name in wanted and wanted[s.name].shape != tuple(s.shape):
             raise ValueError(f"plan lists tensor '{s.name}' twice with different shapes")
         wanted[s.name] = s
-    missing = sorted(n for n in wanted if n not in index)
+    missing = sorted(n for n in wanted if n not in index and not wanted[n].optional)
     unexpected = sorted(n for n in index if n not in wanted)
     wrong_shape, wrong_dtype = [], []
     for n, s in wanted.items():
