@@ -78,28 +78,34 @@ TQ_EXPORT int tq_bias_kv_write(const float* qkv, void* q_out, void* cache, int a
 }
 
 // ---------------------------------------------------------------------------------------
-// The same split with norms and rotations on the way.  Per query and key head, in this order: an RMS norm with a weight
-// shared by the heads (q_norm_w / k_norm_w fp32 [dk], x / sqrt(mean(x^2) + norm_eps) * w; null: none), the rotation
-// by the token's position (the first rot_dims elements of each head, pairs of neighbours or of halves, angle =
-// position * freq[i] in fp32, cos and sin multiplied by `mag`), then a unit norm (unit_eps > 0:
-// x / sqrt(mean(x^2) + unit_eps); 0: left as it is).  Values: kv head g caches value head g / v_share of the row
-// (v_share > 1: neighbouring key heads keep the same values), turned by position * v_freq[m] over all dv elements
-// in the same pairing (v_freq fp32 [dv / 2]; null: as they are).
-// Grid (token, groups of four query and key heads): a warp per head; the blocks of a token share out the copy of the values.
+// The same split with norms and rotations on the way.  Per query and key head, in this order: an RMS norm
+// (q_norm_w / k_norm_w; null: none; x / sqrt(mean(x^2) + norm_eps) * w), either of each head by itself with a weight
+// fp32 [dk] that the heads share, or (norm_rows) of all query heads as one row and all key heads as another with
+// weights fp32 [nh * dk] and [nkv * dk]; the rotation by the token's position (the first rot_dims elements of each head,
+// pairs of neighbours or of halves, angle = position * freq[i] in fp32, cos and sin multiplied by `mag`); a unit norm
+// (unit_eps > 0: x / sqrt(mean(x^2) + unit_eps); 0: left as it is); and for queries a factor that grows with the position
+// (temp_every > 0: 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1)).  Values: kv head g caches value head
+// g / v_share of the row (v_share > 1: neighbouring key heads keep the same values; v_from_k: the row holds no values,
+// key head g / v_share as it leaves the projection is the value, dv == dk), turned by position * v_freq[m] over all dv
+// elements in the same pairing (v_freq fp32 [dv / 2]; null: as they are).
+// A warp per head (warps loop over the heads where the block has fewer); the blocks of a token share out the heads and
+// the copy of the values.  Grid (token, groups of four heads), or with norm_rows (token) with up to sixteen warps.
 // ---------------------------------------------------------------------------------------
+#define BA_ROT_MAX_WARPS 16
 template <typename TA>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(32 * BA_ROT_MAX_WARPS)
 bias_kv_write_rot_kernel(const float* __restrict__ qkv, int row_stride, TA* __restrict__ q_out, TA* __restrict__ cache,
                          const float* __restrict__ freq, int rot_dims, int halves, float mag, float unit_eps,
-                         const float* __restrict__ q_norm_w, const float* __restrict__ k_norm_w, float norm_eps,
-                         const float* __restrict__ v_freq, int v_share,
+                         const float* __restrict__ q_norm_w, const float* __restrict__ k_norm_w, float norm_eps, int norm_rows,
+                         const float* __restrict__ v_freq, int v_share, int v_from_k, float temp_coef, int temp_every,
                          const int* __restrict__ positions, const int* __restrict__ seq_of_token,
                          const int* __restrict__ page_table, int table_stride, int page_size,
                          int nh, int nkv, int dk, int dv, int n_seqs, int n_pages) {
     tq_grid_wait();                    // everything below may read what the previous kernel wrote
     tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
-    __shared__ float s_head[4][BA_MAX_DIM];
-    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    extern __shared__ float s_heads[]; // [warps][dk]
+    __shared__ float scratch[33];
+    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
     const int nq = nh * dk, nk = nkv * dk, nv = nkv * dv, dr = dk + dv;
     const float* row = qkv + (size_t)t * row_stride;
     const int pos = positions[t];
@@ -112,69 +118,106 @@ bias_kv_write_rot_kernel(const float* __restrict__ qkv, int row_stride, TA* __re
     if (cache != nullptr)
         for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < nv; i += gridDim.y * blockDim.x) {
             const int g = i / dv, e = i % dv;
-            const float* vh = row + nq + nk + (size_t)(g / v_share) * dv;
+            const float* vh = row + nq + (v_from_k ? 0 : nk) + (size_t)(g / v_share) * dv;
             const float v = v_freq ? tq_rotated(vh, e, dv & ~1, halves, v_freq, pos) : vh[e];
             cache[(((size_t)page * nkv + g) * page_size + slot) * dr + dk + e] = tq_from_float<TA>(v);
         }
-    const int head = blockIdx.y * 4 + warp;
-    if (head >= nh + nkv || (head >= nh && cache == nullptr)) return;      // without a cache the rows may hold queries only
-    const float* src = row + (size_t)head * dk;                // keys follow the queries in the row
-    float* sh = s_head[warp];
-    const float* nw = head < nh ? q_norm_w : k_norm_w;
-    if (nw != nullptr) {
+    const int last = cache == nullptr ? nh : nh + nkv;         // without a cache the rows may hold queries only
+    float q_rs = 1.f, k_rs = 1.f;
+    if (norm_rows) {                   // the same for the whole block
+        if (q_norm_w != nullptr) {
+            float ss = 0.f;
+            for (int i = threadIdx.x; i < nq; i += blockDim.x) ss += row[i] * row[i];
+            q_rs = 1.0f / sqrtf(tq_block_sum(ss, scratch) / (float)nq + norm_eps);
+        }
+        if (k_norm_w != nullptr && cache != nullptr) {
+            float ss = 0.f;
+            for (int i = threadIdx.x; i < nk; i += blockDim.x) ss += row[nq + i] * row[nq + i];
+            k_rs = 1.0f / sqrtf(tq_block_sum(ss, scratch) / (float)nk + norm_eps);
+        }
+    }
+    float* sh = s_heads + (size_t)warp * dk;
+    for (int head = blockIdx.y * n_warps + warp; head < last; head += gridDim.y * n_warps) {
+        const bool is_q = head < nh;
+        const float* src = row + (size_t)head * dk;            // keys follow the queries in the row
+        const float* nw = is_q ? q_norm_w : k_norm_w;
+        if (nw != nullptr) {
+            float rs = is_q ? q_rs : k_rs;
+            if (norm_rows) {
+                nw += (size_t)(is_q ? head : head - nh) * dk;
+            } else {
+                float ss = 0.f;
+                for (int e = lane; e < dk; e += 32) { const float x = src[e]; ss += x * x; }
+                rs = 1.0f / sqrtf(tq_warp_sum(ss) / (float)dk + norm_eps);
+            }
+            for (int e = lane; e < dk; e += 32) sh[e] = src[e] * rs * nw[e];
+        } else {
+            for (int e = lane; e < dk; e += 32) sh[e] = src[e];
+        }
+        __syncwarp();
+        const int half = rot_dims >> 1;
+        for (int i = lane; i < half; i += 32) {                // a lane turns its pairs in place, one sincos a pair
+            const int a = halves ? i : 2 * i, b = halves ? i + half : 2 * i + 1;
+            float sn, cs;
+            sincosf((float)pos * freq[i], &sn, &cs);
+            const float u = sh[a], v = sh[b];
+            sh[a] = (u * cs - v * sn) * mag;
+            sh[b] = (v * cs + u * sn) * mag;
+        }
+        __syncwarp();
+        float v[BA_EPL];
         float ss = 0.f;
-        for (int e = lane; e < dk; e += 32) { const float x = src[e]; ss += x * x; }
-        const float rs = 1.0f / sqrtf(tq_warp_sum(ss) / (float)dk + norm_eps);
-        for (int e = lane; e < dk; e += 32) sh[e] = src[e] * rs * nw[e];
-    } else {
-        for (int e = lane; e < dk; e += 32) sh[e] = src[e];
-    }
-    __syncwarp();
-    float v[BA_EPL];
-    float ss = 0.f;
 #pragma unroll
-    for (int j = 0; j < BA_EPL; ++j) {
-        const int e = lane + 32 * j;
-        v[j] = e < dk ? tq_rotated(sh, e, rot_dims, halves, freq, pos) * (e < rot_dims ? mag : 1.0f) : 0.f;
-        ss += v[j] * v[j];
-    }
-    float rs = 1.f;
-    if (unit_eps > 0.f) rs = 1.0f / sqrtf(tq_warp_sum(ss) / (float)dk + unit_eps);
-    TA* dst = head < nh ? q_out + ((size_t)t * nh + head) * dk
-                        : (cache ? cache + (((size_t)page * nkv + (head - nh)) * page_size + slot) * dr : nullptr);
-    if (dst == nullptr) return;
+        for (int j = 0; j < BA_EPL; ++j) {
+            const int e = lane + 32 * j;
+            v[j] = e < dk ? sh[e] : 0.f;
+            ss += v[j] * v[j];
+        }
+        float rs = 1.f;
+        if (unit_eps > 0.f) rs = 1.0f / sqrtf(tq_warp_sum(ss) / (float)dk + unit_eps);
+        if (is_q && temp_every > 0) rs *= 1.0f + temp_coef * logf((float)((pos + 1) / temp_every) + 1.0f);
+        TA* dst = is_q ? q_out + ((size_t)t * nh + head) * dk : cache + (((size_t)page * nkv + (head - nh)) * page_size + slot) * dr;
 #pragma unroll
-    for (int j = 0; j < BA_EPL; ++j) {
-        const int e = lane + 32 * j;
-        if (e < dk) dst[e] = tq_from_float<TA>(v[j] * rs);
+        for (int j = 0; j < BA_EPL; ++j) {
+            const int e = lane + 32 * j;
+            if (e < dk) dst[e] = tq_from_float<TA>(v[j] * rs);
+        }
+        __syncwarp();                  // the warp's row in shared memory is free for its next head
     }
 }
 
-// qkv: fp32 rows of row_stride floats that begin with [q | k | v] (v: nkv / v_share heads); freq: fp32 [rot_dims / 2]
-// (null with rot_dims 0).
+// qkv: fp32 rows of row_stride floats that begin with [q | k | v] (v: nkv / v_share heads; none with v_from_k); freq: fp32
+// [rot_dims / 2] (null with rot_dims 0).
 TQ_EXPORT int tq_bias_kv_write_rot(const float* qkv, int row_stride, void* q_out, void* cache, int act_dtype,
                                    const float* freq, int rot_dims, int halves, float mag, float unit_eps,
-                                   const float* q_norm_w, const float* k_norm_w, float norm_eps, const float* v_freq,
-                                   int v_share, const int* positions,
+                                   const float* q_norm_w, const float* k_norm_w, float norm_eps, int norm_rows, const float* v_freq,
+                                   int v_share, int v_from_k, float temp_coef, int temp_every, const int* positions,
                                    const int* seq_of_token, const int* page_table, int table_stride, int page_size,
                                    int T_, int nh, int nkv, int dk, int dv, int n_seqs, int n_pages, cudaStream_t stream) {
     if (T_ == 0) return 0;
     TQ_REQUIRE(nh >= 1 && nkv >= 1 && dk >= 1 && dv >= 1 && dk <= BA_MAX_DIM, "bias_kv_write_rot: bad sizes %d %d %d %d", nh, nkv, dk, dv);
     TQ_REQUIRE(v_share >= 1 && nkv % v_share == 0, "bias_kv_write_rot: %d key heads cannot share values in groups of %d", nkv, v_share);
-    TQ_REQUIRE(row_stride >= nh * dk + (cache ? nkv * dk + nkv / v_share * dv : 0), "bias_kv_write_rot: rows of %d floats do not hold the heads", row_stride);
+    TQ_REQUIRE(!v_from_k || dk == dv, "bias_kv_write_rot: keys of %d elements cannot be values of %d", dk, dv);
+    TQ_REQUIRE(row_stride >= nh * dk + (cache ? nkv * dk + (v_from_k ? 0 : nkv / v_share * dv) : 0), "bias_kv_write_rot: rows of %d floats do not hold the heads", row_stride);
     TQ_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dk && (rot_dims == 0 || freq != nullptr),
                "bias_kv_write_rot: %d rotated elements of a head of %d", rot_dims, dk);
     TQ_REQUIRE(v_freq == nullptr || dv % 2 == 0, "bias_kv_write_rot: values of %d elements cannot be rotated in pairs", dv);
+    TQ_REQUIRE(temp_every >= 0, "bias_kv_write_rot: a temperature that grows every %d positions", temp_every);
+    int warps = 4;
+    if (norm_rows) warps = nh + nkv >= 16 ? 16 : (nh + nkv >= 8 ? 8 : 4);
+    const dim3 grid(T_, norm_rows ? 1 : (nh + nkv + 3) / 4);
+    const size_t smem = (size_t)warps * dk * sizeof(float);
     TQ_DISPATCH(act_dtype, TA,
-        (tq_launch(dim3(T_, (nh + nkv + 3) / 4), 128, 0, stream)(bias_kv_write_rot_kernel<TA>, qkv, row_stride, (TA*)q_out, (TA*)cache, freq, rot_dims,
-            halves, mag, unit_eps, q_norm_w, k_norm_w, norm_eps, v_freq, v_share, positions, seq_of_token, page_table, table_stride, page_size,
-            nh, nkv, dk, dv, n_seqs, n_pages)));
+        (tq_launch(grid, 32 * warps, smem, stream)(bias_kv_write_rot_kernel<TA>, qkv, row_stride, (TA*)q_out, (TA*)cache, freq, rot_dims,
+            halves, mag, unit_eps, q_norm_w, k_norm_w, norm_eps, norm_rows, v_freq, v_share, v_from_k, temp_coef, temp_every, positions,
+            seq_of_token, page_table, table_stride, page_size, nh, nkv, dk, dv, n_seqs, n_pages)));
     TQ_CHECK_LAUNCH("bias_kv_write_rot");
     return 0;
 }
 
 // ---------------------------------------------------------------------------------------
 // What follows the weighted sums of two designs' attention, per (token, head), in fp32:
+//   tq_elements_gate         every element times the sigmoid of its own gate logit
 //   tq_heads_unrotate_gate   a head's output turned back by its own position (pair m by -position * v_freq[m] over all
 //                            dv elements; null: not turned), times sigmoid of the head's gate logit (one per head, from
 //                            a projection's fp32 rows)
@@ -221,6 +264,47 @@ TQ_EXPORT int tq_heads_unrotate_gate(const void* o, int act_dtype, const float* 
         (tq_launch((unsigned)((items + 3) / 4), 128, 0, stream)(heads_unrotate_gate_kernel<TA>, (const TA*)o, gates, gate_stride, gate_off,
             v_freq, halves, positions, (TA*)out, T_, nh, dv)));
     TQ_CHECK_LAUNCH("heads_unrotate_gate");
+    return 0;
+}
+
+// A thread per four elements of a row (vec: rows and gates allow 16-byte reads of the logits).
+template <typename TA>
+__global__ void __launch_bounds__(256)
+elements_gate_kernel(const TA* __restrict__ o, const float* __restrict__ gates, int gate_stride, int gate_off, TA* __restrict__ out,
+                     long long n4, int N, int vec) {
+    tq_grid_wait();                    // everything below may read what the previous kernel wrote
+    tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n4) return;
+    const int per_row = (N + 3) / 4;
+    const long long t = i / per_row;
+    const int c = (int)(i - t * per_row) * 4;
+    const float* z = gates + (size_t)t * gate_stride + gate_off + c;
+    const TA* src = o + (size_t)t * N + c;
+    TA* dst = out + (size_t)t * N + c;
+    float zv[4];
+    if (vec) {
+        const float4 z4 = *reinterpret_cast<const float4*>(z);
+        zv[0] = z4.x; zv[1] = z4.y; zv[2] = z4.z; zv[3] = z4.w;
+    } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) zv[j] = c + j < N ? z[j] : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+        if (c + j < N) dst[j] = tq_from_float<TA>(tq_to_float(src[j]) / (1.0f + expf(-zv[j])));
+}
+
+TQ_EXPORT int tq_elements_gate(const void* o, int act_dtype, const float* gates, int gate_stride, int gate_off, void* out, int T_,
+                               int N, cudaStream_t stream) {
+    if (T_ == 0) return 0;
+    TQ_REQUIRE(N >= 1 && gate_off >= 0 && gate_off + N <= gate_stride, "elements_gate: the gates lie outside their rows");
+    const long long n4 = (long long)T_ * ((N + 3) / 4);
+    const int vec = N % 4 == 0 && gate_stride % 4 == 0 && gate_off % 4 == 0 && ((uintptr_t)gates & 15) == 0;
+    TQ_DISPATCH(act_dtype, TA,
+        (tq_launch((unsigned)((n4 + 255) / 256), 256, 0, stream)(elements_gate_kernel<TA>, (const TA*)o, gates, gate_stride, gate_off,
+            (TA*)out, n4, N, vec)));
+    TQ_CHECK_LAUNCH("elements_gate");
     return 0;
 }
 

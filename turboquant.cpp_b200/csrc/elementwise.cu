@@ -258,41 +258,67 @@ TQ_EXPORT int tq_add_bias(void* x, int x_dtype, const void* bias, int bias_dtype
 
 // ---------------------------------------------------------------------------------------
 // h[t, i] = glu(gu[t, i], gu[t, I + i])   (gate rows first, then up rows; glu: common.cuh, silu(gate) * up by default)
+// bias (optional, fp32 [2I]): added to gate and up first.  Grid (token, pieces of 1,024 elements), four elements a thread
+// (vec: 16-byte reads of fp32 rows).
 // ---------------------------------------------------------------------------------------
+#define GLU_PIECE 1024
 template <typename TI, typename TO>
-__global__ void silu_mul_kernel(const TI* __restrict__ gu, TO* __restrict__ h, int I, TqGlu act) {
+__global__ void __launch_bounds__(GLU_PIECE / 4)
+silu_mul_kernel(const TI* __restrict__ gu, const float* __restrict__ bias, TO* __restrict__ h, int I, int vec, TqGlu act) {
     tq_grid_wait();                    // everything below may read what the previous kernel wrote
     tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
-    const int t = blockIdx.x;
-    const TI* g = gu + (size_t)t * 2 * I;
-    TO* o = h + (size_t)t * I;
-    for (int i = threadIdx.x; i < I; i += blockDim.x) {
-        const float a = tq_to_float(g[i]), b = tq_to_float(g[I + i]);
+    const TI* g = gu + (size_t)blockIdx.x * 2 * I;
+    TO* o = h + (size_t)blockIdx.x * I;
+    if (vec) {
+        const int i = blockIdx.y * GLU_PIECE + 4 * threadIdx.x;
+        if (i >= I) return;
+        float a[4], b[4];
+        const float4 a4 = *reinterpret_cast<const float4*>(g + i), b4 = *reinterpret_cast<const float4*>(g + I + i);
+        a[0] = a4.x; a[1] = a4.y; a[2] = a4.z; a[3] = a4.w;
+        b[0] = b4.x; b[1] = b4.y; b[2] = b4.z; b[3] = b4.w;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            if (bias) { a[j] += bias[i + j]; b[j] += bias[I + i + j]; }
+            a[j] = tq_glu(a[j], b[j], act);
+        }
+        if constexpr (sizeof(TO) == 2) {
+            __nv_bfloat162 p[2] = {__floats2bfloat162_rn(a[0], a[1]), __floats2bfloat162_rn(a[2], a[3])};
+            *reinterpret_cast<uint2*>(o + i) = *reinterpret_cast<uint2*>(p);
+        } else {
+            *reinterpret_cast<float4*>(o + i) = make_float4(a[0], a[1], a[2], a[3]);
+        }
+        return;
+    }
+    for (int i = blockIdx.y * GLU_PIECE + threadIdx.x; i < min(I, (int)(blockIdx.y + 1) * GLU_PIECE); i += blockDim.x) {
+        float a = tq_to_float(g[i]), b = tq_to_float(g[I + i]);
+        if (bias) { a += bias[i]; b += bias[I + i]; }
         o[i] = tq_from_float<TO>(tq_glu(a, b, act));
     }
 }
 
+static int glu_launch(const void* gu, int in_dtype, const float* bias, void* h, int out_dtype, int T_, int I, TqGlu act, cudaStream_t stream) {
+    const int vec = in_dtype == TQ_F32 && I % 4 == 0 && ((uintptr_t)gu & 15) == 0 && ((uintptr_t)h & 15) == 0;
+    const dim3 grid(T_, (I + GLU_PIECE - 1) / GLU_PIECE);
+    TQ_REQUIRE(grid.y <= 65535, "glu_mul: rows of %d elements exceed the grid limit", I);
+    TQ_DISPATCH(in_dtype, TI, TQ_DISPATCH(out_dtype, TO,
+        (tq_launch(grid, GLU_PIECE / 4, 0, stream)(silu_mul_kernel<TI, TO>, (const TI*)gu, bias, (TO*)h, I, vec, act))));
+    TQ_CHECK_LAUNCH("glu_mul");
+    return 0;
+}
+
 // limit <= 0: no caps.  (limit, slope, offset) = (0, 1, 0): silu(gate) * up.
 TQ_EXPORT int tq_glu_mul(const void* gu, int in_dtype, void* h, int out_dtype, int T_, int I, float limit, float slope,
-                         float offset, int kind, cudaStream_t stream) {
+                         float offset, int kind, const float* bias, cudaStream_t stream) {
     if (T_ == 0) return 0;
     TQ_REQUIRE(T_ > 0 && I > 0, "glu_mul: bad sizes T=%d I=%d", T_, I);
     TQ_REQUIRE(kind == TQ_GLU_SIGMOID || kind == TQ_GLU_GELU_TANH, "glu_mul: unknown activation kind %d", kind);
-    const TqGlu act = tq_glu_params(limit, slope, offset, kind);
-    TQ_DISPATCH(in_dtype, TI, TQ_DISPATCH(out_dtype, TO,
-        (tq_launch(T_, 256, 0, stream)(silu_mul_kernel<TI, TO>, (const TI*)gu, (TO*)h, I, act))));
-    TQ_CHECK_LAUNCH("glu_mul");
-    return 0;
+    return glu_launch(gu, in_dtype, bias, h, out_dtype, T_, I, tq_glu_params(limit, slope, offset, kind), stream);
 }
 
 TQ_EXPORT int tq_silu_mul(const void* gu, int in_dtype, void* h, int out_dtype, int T_, int I, cudaStream_t stream) {
     if (T_ == 0) return 0;
     TQ_REQUIRE(T_ > 0 && I > 0, "silu_mul: bad sizes T=%d I=%d", T_, I);
-    const TqGlu act = tq_glu_params(0.f, 1.f, 0.f);
-    TQ_DISPATCH(in_dtype, TI, TQ_DISPATCH(out_dtype, TO,
-        (tq_launch(T_, 256, 0, stream)(silu_mul_kernel<TI, TO>, (const TI*)gu, (TO*)h, I, act))));
-    TQ_CHECK_LAUNCH("silu_mul");
-    return 0;
+    return glu_launch(gu, in_dtype, nullptr, h, out_dtype, T_, I, tq_glu_params(0.f, 1.f, 0.f), stream);
 }
 
 // ---------------------------------------------------------------------------------------
@@ -406,28 +432,30 @@ TQ_EXPORT int tq_embed_pair_rows(const int* tokens, const void* table, const voi
 
 // ---------------------------------------------------------------------------------------
 // Residual sum with the norm on the sub-layer's output: x[r] += y[r] / sqrt(mean(y[r]^2) + eps) * w, in fp32;
-// `copy` (optional) receives the new x in the activation dtype for the products that read it next.
+// `copy` (optional) receives the new x in the activation dtype for the products that read it next.  y_bias (optional,
+// fp32 [H]): y[r] + y_bias stands where y[r] does (the bias of the projection that ends the sub-layer).
 // ---------------------------------------------------------------------------------------
 template <typename TY, typename TW, typename TO>
 __global__ void add_rmsnorm_kernel(float* __restrict__ x, const TY* __restrict__ y, const TW* __restrict__ w,
                                    TO* __restrict__ copy, int H, float eps, const TW* __restrict__ next_w,
-                                   TO* __restrict__ next_out, float next_eps) {
+                                   TO* __restrict__ next_out, float next_eps, const float* __restrict__ y_bias) {
     tq_grid_wait();                    // everything below may read what the previous kernel wrote
     tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
     __shared__ float scratch[33];
     const size_t r = blockIdx.x;
     const TY* yr = y + r * H;
     float* xr = x + r * H;
+    auto value = [&](int i) { return tq_to_float(yr[i]) + (y_bias ? y_bias[i] : 0.f); };
     float ss = 0.f;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
-        const float v = tq_to_float(yr[i]);
+        const float v = value(i);
         ss += v * v;
     }
     ss = tq_block_sum(ss, scratch);
     const float rs = 1.0f / sqrtf(ss / (float)H + eps);
     float s2 = 0.f;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
-        const float v = xr[i] + tq_to_float(yr[i]) * rs * tq_to_float(w[i]);
+        const float v = xr[i] + value(i) * rs * tq_to_float(w[i]);
         xr[i] = v;
         s2 += v * v;
         if (copy) copy[r * H + i] = tq_from_float<TO>(v);
@@ -446,7 +474,7 @@ template <typename TW, typename TO, int NV>
 __global__ void __launch_bounds__(ADDN_THREADS)
 add_rmsnorm_vec_kernel(float* __restrict__ x, const float* __restrict__ y, const TW* __restrict__ w,
                        TO* __restrict__ copy, int H, float eps, const TW* __restrict__ next_w,
-                       TO* __restrict__ next_out, float next_eps) {
+                       TO* __restrict__ next_out, float next_eps, const float* __restrict__ y_bias) {
     tq_grid_wait();                    // everything below may read what the previous kernel wrote
     tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
     __shared__ float scratch[33];
@@ -463,6 +491,12 @@ add_rmsnorm_vec_kernel(float* __restrict__ x, const float* __restrict__ y, const
         if (i < n4) {
             yv[k] = yr[i];
             xv[k] = xr[i];
+            if (y_bias) {
+                yv[k].x += y_bias[4 * i];
+                yv[k].y += y_bias[4 * i + 1];
+                yv[k].z += y_bias[4 * i + 2];
+                yv[k].w += y_bias[4 * i + 3];
+            }
         }
         ss += yv[k].x * yv[k].x + yv[k].y * yv[k].y + yv[k].z * yv[k].z + yv[k].w * yv[k].w;
     }
@@ -508,7 +542,7 @@ add_rmsnorm_vec_kernel(float* __restrict__ x, const float* __restrict__ y, const
 // next_out[r] = x[r] / sqrt(mean(x[r]^2) + next_eps) * next_w, taken in the same pass.
 TQ_EXPORT int tq_add_rmsnorm(float* x, const void* y, int y_dtype, const void* w, int w_dtype, void* copy,
                              int copy_dtype, int R, int H, float eps, const void* next_w, void* next_out, float next_eps,
-                             cudaStream_t stream) {
+                             const float* y_bias, cudaStream_t stream) {
     if (R == 0) return 0;
     TQ_REQUIRE(R > 0 && H > 0, "add_rmsnorm: bad sizes R=%d H=%d", R, H);
     TQ_REQUIRE(next_out == nullptr || next_w != nullptr, "add_rmsnorm: a following norm without its weight%s", "");
@@ -517,7 +551,7 @@ TQ_EXPORT int tq_add_rmsnorm(float* x, const void* y, int y_dtype, const void* w
 #define ADDN_LAUNCH(NV_)                                                                                           \
         TQ_DISPATCH(w_dtype, TW, TQ_DISPATCH(copy_dtype, TO,                                                       \
             (tq_launch(R, ADDN_THREADS, 0, stream)(add_rmsnorm_vec_kernel<TW, TO, NV_>, x, (const float*)y, (const TW*)w, \
-                                                   (TO*)copy, H, eps, (const TW*)next_w, (TO*)next_out, next_eps))))
+                                                   (TO*)copy, H, eps, (const TW*)next_w, (TO*)next_out, next_eps, y_bias))))
         if (nv <= 1) ADDN_LAUNCH(1);
         else if (nv == 2) ADDN_LAUNCH(2);
         else ADDN_LAUNCH(4);
@@ -528,7 +562,7 @@ TQ_EXPORT int tq_add_rmsnorm(float* x, const void* y, int y_dtype, const void* w
     const int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
     TQ_DISPATCH(y_dtype, TY, TQ_DISPATCH(w_dtype, TW, TQ_DISPATCH(copy_dtype, TO,
         (tq_launch(R, threads, 0, stream)(add_rmsnorm_kernel<TY, TW, TO>, x, (const TY*)y, (const TW*)w, (TO*)copy, H,
-                                          eps, (const TW*)next_w, (TO*)next_out, next_eps)))));
+                                          eps, (const TW*)next_w, (TO*)next_out, next_eps, y_bias)))));
     TQ_CHECK_LAUNCH("add_rmsnorm");
     return 0;
 }
@@ -597,18 +631,23 @@ TQ_EXPORT int tq_rotate_pairs(void* x, int dtype, const float* freq, const int* 
 }
 
 // ---------------------------------------------------------------------------------------
-// The mean of two branches, each under an RMS norm of its own:
-//   out[r] = (a[r] / sqrt(mean(a[r]^2) + eps) * wa + b[r] / sqrt(mean(b[r]^2) + eps) * wb) / 2, in fp32.
+// The weighted sum of two branches, each under an RMS norm of its own (fa = fb = 1/2: their mean):
+//   out[r] = fa * a[r] / sqrt(mean(a[r]^2) + eps) * wa + fb * b[r] / sqrt(mean(b[r]^2) + eps) * wb, in fp32.
+// Without the weights (wa and wb null) the branches come as they are: out[r] = fa * a[r] + fb * b[r].
 // ---------------------------------------------------------------------------------------
 template <typename TW>
 __global__ void mean_of_norms_kernel(const float* __restrict__ a, const TW* __restrict__ wa, const float* __restrict__ b,
-                                     const TW* __restrict__ wb, float* __restrict__ out, int H, float eps) {
+                                     const TW* __restrict__ wb, float* __restrict__ out, int H, float eps, float fa, float fb) {
     tq_grid_wait();                    // everything below may read what the previous kernel wrote
     tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
     __shared__ float scratch[33];
     const size_t r = blockIdx.x;
     const float* ar = a + r * H;
     const float* br = b + r * H;
+    if (wa == nullptr) {                           // the same for the whole launch
+        for (int i = threadIdx.x; i < H; i += blockDim.x) out[r * H + i] = fa * ar[i] + fb * br[i];
+        return;
+    }
     float sa = 0.f, sb = 0.f;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
         const float u = ar[i], v = br[i];
@@ -619,24 +658,25 @@ __global__ void mean_of_norms_kernel(const float* __restrict__ a, const TW* __re
     sb = tq_block_sum(sb, scratch);
     const float ra = 1.0f / sqrtf(sa / (float)H + eps), rb = 1.0f / sqrtf(sb / (float)H + eps);
     for (int i = threadIdx.x; i < H; i += blockDim.x)
-        out[r * H + i] = 0.5f * (ar[i] * ra * tq_to_float(wa[i]) + br[i] * rb * tq_to_float(wb[i]));
+        out[r * H + i] = fa * (ar[i] * ra * tq_to_float(wa[i])) + fb * (br[i] * rb * tq_to_float(wb[i]));
 }
 
 TQ_EXPORT int tq_mean_of_norms(const float* a, const void* wa, const float* b, const void* wb, int w_dtype, float* out,
-                               int R, int H, float eps, cudaStream_t stream) {
+                               int R, int H, float eps, float fa, float fb, cudaStream_t stream) {
     if (R == 0) return 0;
+    TQ_REQUIRE((wa == nullptr) == (wb == nullptr), "mean_of_norms: both branches have a norm or neither%s", "");
     TQ_REQUIRE(R > 0 && H > 0, "mean_of_norms: bad sizes R=%d H=%d", R, H);
     const int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
     TQ_DISPATCH(w_dtype, TW,
-        (tq_launch(R, threads, 0, stream)(mean_of_norms_kernel<TW>, a, (const TW*)wa, b, (const TW*)wb, out, H, eps)));
+        (tq_launch(R, threads, 0, stream)(mean_of_norms_kernel<TW>, a, (const TW*)wa, b, (const TW*)wb, out, H, eps, fa, fb)));
     TQ_CHECK_LAUNCH("mean_of_norms");
     return 0;
 }
 
 // ---------------------------------------------------------------------------------------
-// The mean of two normed branches under a further norm, summed into the stream, with the norm that reads the stream
-// next (optional) in the same pass:
-//   m[r] = (a[r] / sqrt(mean(a[r]^2) + pair_eps) * wa + b[r] / sqrt(mean(b[r]^2) + pair_eps) * wb) / 2
+// The weighted sum of two branches, normed or (wa and wb null) as they are, under a further norm, summed into the
+// stream, with the norm that reads the stream next (optional) in the same pass:
+//   m[r] = fa * a[r] / sqrt(mean(a[r]^2) + pair_eps) * wa + fb * b[r] / sqrt(mean(b[r]^2) + pair_eps) * wb
 //   x[r] += m[r] / sqrt(mean(m[r]^2) + eps) * w;   next_out[r] = x[r] / sqrt(mean(x[r]^2) + next_eps) * next_w
 // all in fp32.  The vector form keeps a thread's float4 pieces of the row in registers from the first sums to the last
 // output (rows of a multiple of four, up to 4 * ADDN_THREADS * NV elements); the plain form reads the row again.
@@ -646,7 +686,7 @@ __global__ void __launch_bounds__(ADDN_THREADS)
 add_rmsnorm_pair_vec_kernel(float* __restrict__ x, const float* __restrict__ a, const TW* __restrict__ wa,
                             const float* __restrict__ b, const TW* __restrict__ wb, float pair_eps,
                             const TW* __restrict__ w, TO* __restrict__ copy, int H, float eps,
-                            const TW* __restrict__ next_w, TO* __restrict__ next_out, float next_eps) {
+                            const TW* __restrict__ next_w, TO* __restrict__ next_out, float next_eps, float fa, float fb) {
     tq_grid_wait();                    // everything below may read what the previous kernel wrote
     tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
     __shared__ float scratch[33];
@@ -669,19 +709,24 @@ add_rmsnorm_pair_vec_kernel(float* __restrict__ x, const float* __restrict__ a, 
         sa += av[k].x * av[k].x + av[k].y * av[k].y + av[k].z * av[k].z + av[k].w * av[k].w;
         sb += bv[k].x * bv[k].x + bv[k].y * bv[k].y + bv[k].z * bv[k].z + bv[k].w * bv[k].w;
     }
-    sa = tq_block_sum(sa, scratch);
-    sb = tq_block_sum(sb, scratch);
-    const float ra = 1.0f / sqrtf(sa / (float)H + pair_eps), rb = 1.0f / sqrtf(sb / (float)H + pair_eps);
+    float ra = fa, rb = fb;
+    if (wa) {                                      // the same for the whole launch
+        sa = tq_block_sum(sa, scratch);
+        sb = tq_block_sum(sb, scratch);
+        ra = fa / sqrtf(sa / (float)H + pair_eps);
+        rb = fb / sqrtf(sb / (float)H + pair_eps);
+    }
+    auto wt = [](const TW* p, int i) { return p ? tq_to_float(p[i]) : 1.0f; };
     float sm = 0.f;
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
         const int i = threadIdx.x + k * ADDN_THREADS;
         if (i < n4) {
             float4 m;
-            m.x = 0.5f * (av[k].x * ra * tq_to_float(wa[4 * i]) + bv[k].x * rb * tq_to_float(wb[4 * i]));
-            m.y = 0.5f * (av[k].y * ra * tq_to_float(wa[4 * i + 1]) + bv[k].y * rb * tq_to_float(wb[4 * i + 1]));
-            m.z = 0.5f * (av[k].z * ra * tq_to_float(wa[4 * i + 2]) + bv[k].z * rb * tq_to_float(wb[4 * i + 2]));
-            m.w = 0.5f * (av[k].w * ra * tq_to_float(wa[4 * i + 3]) + bv[k].w * rb * tq_to_float(wb[4 * i + 3]));
+            m.x = av[k].x * ra * wt(wa, 4 * i) + bv[k].x * rb * wt(wb, 4 * i);
+            m.y = av[k].y * ra * wt(wa, 4 * i + 1) + bv[k].y * rb * wt(wb, 4 * i + 1);
+            m.z = av[k].z * ra * wt(wa, 4 * i + 2) + bv[k].z * rb * wt(wb, 4 * i + 2);
+            m.w = av[k].w * ra * wt(wa, 4 * i + 3) + bv[k].w * rb * wt(wb, 4 * i + 3);
             av[k] = m;
             sm += m.x * m.x + m.y * m.y + m.z * m.z + m.w * m.w;
         }
@@ -728,7 +773,7 @@ template <typename TW, typename TO>
 __global__ void add_rmsnorm_pair_kernel(float* __restrict__ x, const float* __restrict__ a, const TW* __restrict__ wa,
                                         const float* __restrict__ b, const TW* __restrict__ wb, float pair_eps,
                                         const TW* __restrict__ w, TO* __restrict__ copy, int H, float eps,
-                                        const TW* __restrict__ next_w, TO* __restrict__ next_out, float next_eps) {
+                                        const TW* __restrict__ next_w, TO* __restrict__ next_out, float next_eps, float fa, float fb) {
     tq_grid_wait();                    // everything below may read what the previous kernel wrote
     tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
     __shared__ float scratch[33];
@@ -741,10 +786,14 @@ __global__ void add_rmsnorm_pair_kernel(float* __restrict__ x, const float* __re
         sa += ar[i] * ar[i];
         sb += br[i] * br[i];
     }
-    sa = tq_block_sum(sa, scratch);
-    sb = tq_block_sum(sb, scratch);
-    const float ra = 1.0f / sqrtf(sa / (float)H + pair_eps), rb = 1.0f / sqrtf(sb / (float)H + pair_eps);
-    auto mean = [&](int i) { return 0.5f * (ar[i] * ra * tq_to_float(wa[i]) + br[i] * rb * tq_to_float(wb[i])); };
+    float ra = fa, rb = fb;
+    if (wa) {                                      // the same for the whole launch
+        sa = tq_block_sum(sa, scratch);
+        sb = tq_block_sum(sb, scratch);
+        ra = fa / sqrtf(sa / (float)H + pair_eps);
+        rb = fb / sqrtf(sb / (float)H + pair_eps);
+    }
+    auto mean = [&](int i) { return ar[i] * ra * (wa ? tq_to_float(wa[i]) : 1.0f) + br[i] * rb * (wb ? tq_to_float(wb[i]) : 1.0f); };
     float sm = 0.f;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
         const float m = mean(i);
@@ -769,8 +818,9 @@ __global__ void add_rmsnorm_pair_kernel(float* __restrict__ x, const float* __re
 // wa, wb, w and next_w share one dtype; copy and next_out another.
 TQ_EXPORT int tq_add_rmsnorm_pair(float* x, const float* a, const void* wa, const float* b, const void* wb, float pair_eps,
                                   const void* w, int w_dtype, void* copy, int copy_dtype, int R, int H, float eps,
-                                  const void* next_w, void* next_out, float next_eps, cudaStream_t stream) {
+                                  const void* next_w, void* next_out, float next_eps, float fa, float fb, cudaStream_t stream) {
     if (R == 0) return 0;
+    TQ_REQUIRE((wa == nullptr) == (wb == nullptr), "add_rmsnorm_pair: both branches have a norm or neither%s", "");
     TQ_REQUIRE(R > 0 && H > 0, "add_rmsnorm_pair: bad sizes R=%d H=%d", R, H);
     TQ_REQUIRE(next_out == nullptr || next_w != nullptr, "add_rmsnorm_pair: a following norm without its weight%s", "");
     if (H % 4 == 0 && H <= 4 * ADDN_THREADS * 4 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)a % 16) == 0 && ((uintptr_t)b % 16) == 0) {
@@ -778,7 +828,7 @@ TQ_EXPORT int tq_add_rmsnorm_pair(float* x, const float* a, const void* wa, cons
 #define ADDP_LAUNCH(NV_)                                                                                           \
         TQ_DISPATCH(w_dtype, TW, TQ_DISPATCH(copy_dtype, TO,                                                       \
             (tq_launch(R, ADDN_THREADS, 0, stream)(add_rmsnorm_pair_vec_kernel<TW, TO, NV_>, x, a, (const TW*)wa, b, \
-                (const TW*)wb, pair_eps, (const TW*)w, (TO*)copy, H, eps, (const TW*)next_w, (TO*)next_out, next_eps))))
+                (const TW*)wb, pair_eps, (const TW*)w, (TO*)copy, H, eps, (const TW*)next_w, (TO*)next_out, next_eps, fa, fb))))
         if (nv <= 1) ADDP_LAUNCH(1);
         else if (nv == 2) ADDP_LAUNCH(2);
         else ADDP_LAUNCH(4);
@@ -789,7 +839,7 @@ TQ_EXPORT int tq_add_rmsnorm_pair(float* x, const float* a, const void* wa, cons
     const int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
     TQ_DISPATCH(w_dtype, TW, TQ_DISPATCH(copy_dtype, TO,
         (tq_launch(R, threads, 0, stream)(add_rmsnorm_pair_kernel<TW, TO>, x, a, (const TW*)wa, b, (const TW*)wb, pair_eps,
-                                          (const TW*)w, (TO*)copy, H, eps, (const TW*)next_w, (TO*)next_out, next_eps))));
+                                          (const TW*)w, (TO*)copy, H, eps, (const TW*)next_w, (TO*)next_out, next_eps, fa, fb))));
     TQ_CHECK_LAUNCH("add_rmsnorm_pair");
     return 0;
 }

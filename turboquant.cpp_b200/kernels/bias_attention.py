@@ -45,31 +45,38 @@ def kv_write_rot(qkv: torch.Tensor, q_out: torch.Tensor, cache: Optional[torch.T
                  rot_dims: int, halves: bool, unit_eps: float, positions: torch.Tensor, seq_of_token: torch.Tensor,
                  page_table: torch.Tensor, page_size: int, heads: int, kv_heads: int, dk: int, dv: int, mag: float = 1.0,
                  q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None, norm_eps: float = 0.0,
-                 v_freq: Optional[torch.Tensor] = None, v_share: int = 1) -> None:
+                 v_freq: Optional[torch.Tensor] = None, v_share: int = 1, norm_rows: bool = False, values_are_keys: bool = False,
+                 temperature: Optional[tuple] = None) -> None:
     """The split of `kv_write` with norms and rotations on the way.  qkv float32 [T, >= heads*dk + kv_heads*dk +
     (kv_heads / v_share)*dv]: rows that begin with [q | k | v] (they may hold more behind).  Per query and key head:
-    with q_norm / k_norm (float32 [dk], shared by the heads) the head becomes x / sqrt(mean(x^2) + norm_eps) * weight;
+    with q_norm / k_norm (float32 [dk], shared by the heads) the head becomes x / sqrt(mean(x^2) + norm_eps) * weight
+    (norm_rows: the mean is taken over all query heads, or all key heads, and the weights are [heads * dk] and [kv_heads * dk]);
     then the first rot_dims elements turn by position * freq[i] (freq float32 [rot_dims / 2]; pairs (2i, 2i+1), or
     (i, i + rot_dims/2) with `halves`), cos and sin multiplied by `mag`; then, with unit_eps > 0, each head is divided
-    by sqrt(mean(head^2) + unit_eps).  Queries go to q_out [T, heads, dk], keys and values to the token's place in
+    by sqrt(mean(head^2) + unit_eps); then, with temperature (coef, every), queries are multiplied by
+    1 + coef * ln(floor((position + 1) / every) + 1).  Queries go to q_out [T, heads, dk], keys and values to the token's place in
     cache [pages, 1, kv_heads, page_size, dk + dv]; key head g keeps value head g // v_share of the row, turned by
-    position * v_freq[m] over all dv elements in the same pairing where v_freq (float32 [dv / 2]) is given.  Without a
+    position * v_freq[m] over all dv elements in the same pairing where v_freq (float32 [dv / 2]) is given.
+    values_are_keys: the row is [q | k] and a key as it leaves the projection is the value as well.  Without a
     cache the rows need to hold the queries only."""
     want_f32(qkv, "the fused projection")
     want_int32(positions, "positions")
     T = qkv.shape[0]
     if v_share < 1 or kv_heads % v_share or \
-            qkv.shape[1] < heads * dk + (kv_heads * dk + kv_heads // v_share * dv if cache is not None else 0):
+            qkv.shape[1] < heads * dk + (kv_heads * dk + (0 if values_are_keys else kv_heads // v_share * dv) if cache is not None else 0):
         raise KernelError("kv_write_rot: the projection's width does not hold the heads")
     if freq is not None:
         want_f32(freq, "frequencies")
         if 2 * freq.numel() != rot_dims:
             raise KernelError("kv_write_rot: one frequency per rotated pair")
-    for w in (q_norm, k_norm):
+    for w, n in ((q_norm, heads), (k_norm, kv_heads)):
         if w is not None:
             want_f32(w, "a head norm's weight")
-            if w.numel() != dk:
-                raise KernelError("kv_write_rot: a head norm's weight has one element per element of a head")
+            if w.numel() != (n * dk if norm_rows else dk):
+                raise KernelError("kv_write_rot: a norm's weight has one element per element of what it is taken over")
+    coef, every = temperature if temperature is not None else (0.0, 0)
+    if temperature is not None and every < 1:
+        raise KernelError("kv_write_rot: the temperature grows every so many positions, at least every one")
     if v_freq is not None:
         want_f32(v_freq, "the values' frequencies")
         if 2 * v_freq.numel() != dv:
@@ -80,8 +87,8 @@ def kv_write_rot(qkv: torch.Tensor, q_out: torch.Tensor, cache: Optional[torch.T
     lib = load_kernel(_LIB)
     check(_LIB, lib.tq_bias_kv_write_rot(
         ptr(qkv), c_int(qkv.shape[1]), ptr(q_out), ptr(cache), c_int(code(q_out.dtype)), ptr(freq), c_int(rot_dims),
-        c_int(1 if halves else 0), c_float(mag), c_float(unit_eps), ptr(q_norm), ptr(k_norm), c_float(norm_eps), ptr(v_freq),
-        c_int(v_share), ptr(positions), ptr(seq_of_token), ptr(page_table),
+        c_int(1 if halves else 0), c_float(mag), c_float(unit_eps), ptr(q_norm), ptr(k_norm), c_float(norm_eps),
+        c_int(1 if norm_rows else 0), ptr(v_freq), c_int(v_share), c_int(1 if values_are_keys else 0), c_float(coef), c_int(every), ptr(positions), ptr(seq_of_token), ptr(page_table),
         c_int(page_table.shape[1]), c_int(page_size), c_int(T), c_int(heads), c_int(kv_heads), c_int(dk), c_int(dv),
         c_int(page_table.shape[0]), c_int(cache.shape[0] if cache is not None else 0), stream()))
 
@@ -104,6 +111,19 @@ def heads_unrotate_gate(o: torch.Tensor, gates: torch.Tensor, gate_off: int, v_f
     check(_LIB, lib.tq_heads_unrotate_gate(ptr(o), c_int(code(o.dtype)), ptr(gates), c_int(gates.shape[1]), c_int(gate_off),
                                            ptr(v_freq), c_int(1 if halves else 0), ptr(positions), ptr(out), c_int(T),
                                            c_int(heads), c_int(dv), stream()))
+    return out
+
+
+def elements_gate(o: torch.Tensor, gates: torch.Tensor, gate_off: int, out: torch.Tensor) -> torch.Tensor:
+    """out[t, i] = o[t, i] * sigmoid(gates[t, gate_off + i]).  o, out [T, N] in the activation dtype (they may be the same
+    tensor); gates float32 rows."""
+    want_f32(gates, "the gates")
+    T, N = o.shape
+    if out.shape != o.shape or out.dtype != o.dtype or gates.shape[0] != T:
+        raise KernelError("elements_gate: input, gates and output must have the same rows, input and output one dtype")
+    lib = load_kernel(_LIB)
+    check(_LIB, lib.tq_elements_gate(ptr(o), c_int(code(o.dtype)), ptr(gates), c_int(gates.shape[1]), c_int(gate_off), ptr(out),
+                                     c_int(T), c_int(N), stream()))
     return out
 
 

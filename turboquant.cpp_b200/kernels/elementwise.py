@@ -91,28 +91,33 @@ SILU_GLU = Glu()
 GELU_TANH_GLU = Glu(kind=GLU_GELU_TANH)
 
 
-def glu_mul(gate_up: torch.Tensor, out: torch.Tensor, glu: Glu = SILU_GLU) -> torch.Tensor:
-    """out[t, i] = glu(gate_up[t, i], gate_up[t, I + i]), computed in float32."""
+def glu_mul(gate_up: torch.Tensor, out: torch.Tensor, glu: Glu = SILU_GLU, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out[t, i] = glu(gate_up[t, i], gate_up[t, I + i]), computed in float32; bias float32 [2I]: added to gate and up first."""
     T, I = out.shape
+    if bias is not None:
+        want_f32(bias, "the bias")
+        if bias.numel() != 2 * I:
+            raise KernelError("glu_mul: one bias per element of gate and up")
     lib = load_kernel(_LIB)
     check(_LIB, lib.tq_glu_mul(ptr(gate_up), c_int(code(gate_up.dtype)), ptr(out), c_int(code(out.dtype)),
                                c_int(T), c_int(I), c_float(glu.limit), c_float(glu.slope), c_float(glu.offset),
-                               c_int(glu.kind), stream()))
+                               c_int(glu.kind), ptr(bias), stream()))
     return out
 
 
-def mean_of_norms(a: torch.Tensor, wa: torch.Tensor, b: torch.Tensor, wb: torch.Tensor, eps: float,
-                  out: torch.Tensor) -> torch.Tensor:
-    """out = (a / rms(a) * wa + b / rms(b) * wb) / 2 row by row in float32: two branches, each under an RMS norm of its
-    own, averaged.  a, b, out float32 [R, H]."""
+def mean_of_norms(a: torch.Tensor, wa: Optional[torch.Tensor], b: torch.Tensor, wb: Optional[torch.Tensor], eps: float,
+                  out: torch.Tensor, factors=(0.5, 0.5)) -> torch.Tensor:
+    """out = fa * a / rms(a) * wa + fb * b / rms(b) * wb row by row in float32: two branches, each under an RMS norm of
+    its own, averaged (or added with other factors).  Without weights (both None) the branches come as they are.
+    a, b, out float32 [R, H]."""
     for t, what in ((a, "the first branch"), (b, "the second branch"), (out, "the mean")):
         want_f32(t, what)
-    if a.shape != b.shape or out.shape != a.shape or wa.dtype != wb.dtype:
+    if a.shape != b.shape or out.shape != a.shape or (wa is None) != (wb is None) or (wa is not None and wa.dtype != wb.dtype):
         raise KernelError("mean_of_norms: the branches, their weights and the output must agree")
     R, H = a.shape
     lib = load_kernel(_LIB)
-    check(_LIB, lib.tq_mean_of_norms(ptr(a), ptr(wa), ptr(b), ptr(wb), c_int(code(wa.dtype)), ptr(out), c_int(R), c_int(H),
-                                     c_float(eps), stream()))
+    check(_LIB, lib.tq_mean_of_norms(ptr(a), ptr(wa), ptr(b), ptr(wb), c_int(code(wa.dtype) if wa is not None else 0), ptr(out),
+                                     c_int(R), c_int(H), c_float(eps), c_float(factors[0]), c_float(factors[1]), stream()))
     return out
 
 
@@ -183,13 +188,18 @@ def embed_pair_rows(tokens: torch.Tensor, table: torch.Tensor, pair: Optional[to
 
 def add_rmsnorm(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float,
                 copy: Optional[torch.Tensor] = None, next_weight: Optional[torch.Tensor] = None,
-                next_out: Optional[torch.Tensor] = None, next_eps: Optional[float] = None) -> torch.Tensor:
+                next_out: Optional[torch.Tensor] = None, next_eps: Optional[float] = None,
+                y_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """x += y / sqrt(mean(y^2) + eps) * weight, row by row in float32 (the norm sits on the sub-layer's output);
     `copy` receives the new x in its own dtype.  next_weight, next_out: the norm that reads the new x next is taken
     in the same pass, next_out = x / sqrt(mean(x^2) + next_eps) * next_weight (next_weight in weight's dtype,
-    next_out in copy's if both are given)."""
+    next_out in copy's if both are given).  y_bias float32 [H]: y + y_bias stands where y does."""
     want_f32(x, "the residual stream")
     R, H = x.shape
+    if y_bias is not None:
+        want_f32(y_bias, "the sub-layer's bias")
+        if y_bias.numel() != H:
+            raise KernelError("add_rmsnorm: the sub-layer's bias must have the norm's size")
     if next_out is not None:
         if next_weight is None or next_weight.dtype != weight.dtype or (copy is not None and copy.dtype != next_out.dtype):
             raise KernelError("add_rmsnorm: the following norm's weight and output must share the dtypes of weight and copy")
@@ -198,16 +208,16 @@ def add_rmsnorm(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: flo
     check(_LIB, lib.tq_add_rmsnorm(ptr(x), ptr(y), c_int(code(y.dtype)), ptr(weight), c_int(code(weight.dtype)),
                                    ptr(copy), c_int(code(side.dtype) if side is not None else 0), c_int(R), c_int(H),
                                    c_float(eps), ptr(next_weight if next_out is not None else None), ptr(next_out),
-                                   c_float(eps if next_eps is None else next_eps), stream()))
+                                   c_float(eps if next_eps is None else next_eps), ptr(y_bias), stream()))
     return x
 
 
-def add_rmsnorm_pair(x: torch.Tensor, a: torch.Tensor, wa: torch.Tensor, b: torch.Tensor, wb: torch.Tensor, pair_eps: float,
+def add_rmsnorm_pair(x: torch.Tensor, a: torch.Tensor, wa: Optional[torch.Tensor], b: torch.Tensor, wb: Optional[torch.Tensor], pair_eps: float,
                      weight: torch.Tensor, eps: float, copy: Optional[torch.Tensor] = None,
                      next_weight: Optional[torch.Tensor] = None, next_out: Optional[torch.Tensor] = None,
-                     next_eps: Optional[float] = None) -> torch.Tensor:
-    """`mean_of_norms(a, wa, b, wb, pair_eps)` under `add_rmsnorm(x, ., weight, eps, copy, next...)` in one pass:
-    x += m / sqrt(mean(m^2) + eps) * weight with m the mean of the two normed branches.  a, b float32 [R, H]; the four
+                     next_eps: Optional[float] = None, factors=(0.5, 0.5)) -> torch.Tensor:
+    """`mean_of_norms(a, wa, b, wb, pair_eps, factors=)` under `add_rmsnorm(x, ., weight, eps, copy, next...)` in one pass:
+    x += m / sqrt(mean(m^2) + eps) * weight with m the weighted sum of the two branches.  a, b float32 [R, H]; the
     weights share a dtype."""
     want_f32(x, "the residual stream")
     want_f32(a, "the first branch")
@@ -215,7 +225,7 @@ def add_rmsnorm_pair(x: torch.Tensor, a: torch.Tensor, wa: torch.Tensor, b: torc
     R, H = x.shape
     if a.shape != x.shape or b.shape != x.shape:
         raise KernelError("add_rmsnorm_pair: the branches and the stream must agree in shape")
-    ws = [wa, wb, weight] + ([next_weight] if next_out is not None else [])
+    ws = ([wa, wb] if wa is not None or wb is not None else []) + [weight] + ([next_weight] if next_out is not None else [])
     if any(w is None or w.dtype != weight.dtype for w in ws):
         raise KernelError("add_rmsnorm_pair: the norms' weights must share a dtype")
     if next_out is not None and copy is not None and copy.dtype != next_out.dtype:
@@ -225,7 +235,8 @@ def add_rmsnorm_pair(x: torch.Tensor, a: torch.Tensor, wa: torch.Tensor, b: torc
     check(_LIB, lib.tq_add_rmsnorm_pair(ptr(x), ptr(a), ptr(wa), ptr(b), ptr(wb), c_float(pair_eps), ptr(weight),
                                         c_int(code(weight.dtype)), ptr(copy), c_int(code(side.dtype) if side is not None else 0),
                                         c_int(R), c_int(H), c_float(eps), ptr(next_weight if next_out is not None else None),
-                                        ptr(next_out), c_float(eps if next_eps is None else next_eps), stream()))
+                                        ptr(next_out), c_float(eps if next_eps is None else next_eps), c_float(factors[0]), c_float(factors[1]),
+                                        stream()))
     return x
 
 

@@ -35,6 +35,24 @@ def conv_silu(proj: torch.Tensor, off: int, weight: torch.Tensor, bias: Optional
     return out
 
 
+def conv_silu_step(proj: torch.Tensor, off: int, weight: torch.Tensor, bias: Optional[torch.Tensor], kept: torch.Tensor,
+                   out: torch.Tensor, slots: torch.Tensor) -> torch.Tensor:
+    """`conv_silu` for steps in which every sequence brings one token (token t is sequence t), in one launch."""
+    want_f32(proj, "the projection")
+    want_f32(out, "the convolution's output")
+    want_f32(kept, "the kept inputs")
+    want_int32(slots, "slots")
+    T, C = out.shape
+    taps = weight.shape[1]
+    if weight.shape[0] != C or kept.shape[1:] != (taps - 1, C) or kept.stride(2) != 1 or kept.stride(1) != C or slots.numel() != T:
+        raise KernelError("conv_silu_step: weight, kept inputs, output and slots do not fit together")
+    lib = load_kernel(_LIB)
+    check(_LIB, lib.tq_conv_silu_step(ptr(proj), c_int(proj.shape[1]), c_int(off), ptr(weight), ptr(bias), c_int(code(weight.dtype)),
+                                      ctypes_ptr(kept), c_longlong(kept.stride(0)), ptr(out), c_int(T), c_int(C), c_int(taps),
+                                      ptr(slots), stream()))
+    return out
+
+
 def ssm_scan(xbc: torch.Tensor, proj: Optional[torch.Tensor], dt_off: int, dt_bias: Optional[torch.Tensor],
              a_log: Optional[torch.Tensor], d_skip: Optional[torch.Tensor], state: torch.Tensor, y: Optional[torch.Tensor], heads: int,
              vdim: int, n_state: int, groups: int, cu_seqlens: torch.Tensor, slots: torch.Tensor,
@@ -104,18 +122,28 @@ def retention_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, ou
 
 
 def gated_group_norm(y: torch.Tensor, proj: torch.Tensor, z_off: int, weight: Optional[torch.Tensor], norm_groups: int,
-                     eps: float, out: torch.Tensor, gate_after: bool = False, sigmoid_gate: bool = False) -> torch.Tensor:
+                     eps: float, out: torch.Tensor, gate_after: bool = False, sigmoid_gate: bool = False,
+                     dots: Optional[torch.Tensor] = None, tops: Optional[torch.Tensor] = None, dot_scale: float = 1.0,
+                     floor: float = 0.0) -> torch.Tensor:
     """out = rms_in_groups(y * silu(z)) * weight with z = proj[:, z_off:z_off+inner]: the gate first, then each of
     the norm_groups equal parts of a row divided by its own root mean square.  gate_after: the norm first, then the
-    gate: rms_in_groups(y) * weight * silu(z).  weight None: no weight.  sigmoid_gate: sigmoid(z) where silu(z) stands."""
+    gate: rms_in_groups(y) * weight * silu(z).  weight None: no weight.  sigmoid_gate: sigmoid(z) where silu(z) stands.
+    dots, tops float32 [T, norm_groups]: part g of y is first multiplied by
+    dot_scale / (max(|dot_scale * dots[t, g]|, exp(-tops[t, g])) + floor)."""
     want_f32(y, "the recurrence's output")
     want_f32(proj, "the projection")
     T, inner = y.shape
+    if dots is not None:
+        want_f32(dots, "the parts' dot products")
+        want_f32(tops, "the parts' maxima")
+        if dots.numel() != T * norm_groups or tops.numel() != T * norm_groups:
+            raise KernelError("gated_group_norm: one dot product and one maximum per token and part")
     lib = load_kernel(_LIB)
     check(_LIB, lib.tq_gated_group_norm(ptr(y), ptr(proj), c_int(proj.shape[1]), c_int(z_off), ptr(weight),
                                         c_int(code(weight.dtype) if weight is not None else 0), ptr(out),
                                         c_int(code(out.dtype)), c_int(T), c_int(inner), c_int(norm_groups), c_float(eps),
-                                        c_int(1 if gate_after else 0), c_int(1 if sigmoid_gate else 0), stream()))
+                                        c_int(1 if gate_after else 0), c_int(1 if sigmoid_gate else 0), ptr(dots), ptr(tops),
+                                        c_float(dot_scale), c_float(floor), stream()))
     return out
 
 
@@ -167,12 +195,20 @@ def retention_step(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off
     return out
 
 
+def _decays_per_head(what: str, dt_bias: torch.Tensor, a_log: torch.Tensor, heads: int, dk: int) -> int:
+    """Decays a head of the delta rule has: dk (a bias per head and key channel) or one (a bias per head)."""
+    if a_log.numel() != heads or dt_bias.numel() not in (heads, heads * dk):
+        raise KernelError(f"{what}: one rate per head, and a decay bias per head or per head and key channel")
+    return dt_bias.numel() // heads
+
+
 def delta_scan(xqkv: torch.Tensor, q_off: int, k_off: int, v_off: int, proj: torch.Tensor, b_off: int, a_raw: torch.Tensor,
                a_off: int, dt_bias: torch.Tensor, a_log: torch.Tensor, state: torch.Tensor, y: torch.Tensor, heads: int,
                kv_heads: int, dk: int, dv: int, unit_eps: float, q_scale: float, cu_seqlens: torch.Tensor,
                slots: torch.Tensor) -> torch.Tensor:
     """The delta rule with a decay per key channel over every sequence's run of new tokens:
     S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; y = S^T q, with k and q made unit vectors
+    (dt_bias of heads elements instead of heads * dk: one decay per head, raw decays a_raw[:, a_off : a_off + heads])
     (x / sqrt(sum(x^2) + unit_eps), q times q_scale), beta = sigmoid(proj[:, b_off + a]) and
     g = exp(-exp(a_log[a]) * softplus(a_raw[:, a_off + a*dk : ...] + dt_bias[a])).  xqkv float32 [T, C] holds q, k
     (kv_heads x dk) and v (heads x dv) from the given columns; state float32 [max_slots, heads, dv, dk] (a head's
@@ -184,11 +220,12 @@ def delta_scan(xqkv: torch.Tensor, q_off: int, k_off: int, v_off: int, proj: tor
     want_int32(slots, "slots")
     if tuple(state.shape[1:]) != (heads, dv, dk) or not state[0].is_contiguous():
         raise KernelError("delta_scan: the state must be [slots, heads, vdim, dim] with dense rows")
-    if dt_bias.numel() != heads * dk or a_log.numel() != heads or y.shape != (xqkv.shape[0], heads * dv):
-        raise KernelError("delta_scan: one decay bias per head and key channel, one rate per head, an output of heads*dv")
+    dper = _decays_per_head("delta_scan", dt_bias, a_log, heads, dk)
+    if y.shape != (xqkv.shape[0], heads * dv):
+        raise KernelError("delta_scan: an output of heads*dv")
     lib = load_kernel(_LIB)
     check(_LIB, lib.tq_delta_scan(ptr(xqkv), c_int(xqkv.shape[1]), c_int(q_off), c_int(k_off), c_int(v_off), ptr(proj),
-                                  c_int(proj.shape[1]), c_int(b_off), ptr(a_raw), c_int(a_raw.shape[1]), c_int(a_off),
+                                  c_int(proj.shape[1]), c_int(b_off), ptr(a_raw), c_int(a_raw.shape[1]), c_int(a_off), c_int(dper),
                                   ptr(dt_bias), ptr(a_log), ctypes_ptr(state), c_longlong(state.stride(0)), ptr(y),
                                   c_int(cu_seqlens.shape[0] - 1), c_int(heads), c_int(kv_heads), c_int(dk), c_int(dv),
                                   c_float(unit_eps), c_float(q_scale), ptr(cu_seqlens), ptr(slots), stream()))
@@ -210,14 +247,128 @@ def delta_scan_runs(xqkv: torch.Tensor, q_off: int, k_off: int, v_off: int, proj
     want_int32(slots, "slots")
     if tuple(state.shape[1:]) != (heads, dv, dk) or not state[0].is_contiguous():
         raise KernelError("delta_scan_runs: the state must be [slots, heads, vdim, dim] with dense rows")
-    if dt_bias.numel() != heads * dk or a_log.numel() != heads or y.shape != (xqkv.shape[0], heads * dv):
-        raise KernelError("delta_scan_runs: one decay bias per head and key channel, one rate per head, an output of heads*dv")
+    dper = _decays_per_head("delta_scan_runs", dt_bias, a_log, heads, dk)
+    if y.shape != (xqkv.shape[0], heads * dv):
+        raise KernelError("delta_scan_runs: an output of heads*dv")
     lib = load_kernel(_LIB)
     T = xqkv.shape[0]
-    rows = torch.empty((T, int(lib.tq_delta_rows_width(c_int(heads), c_int(kv_heads), c_int(dk)))), dtype=torch.float32, device=xqkv.device)
+    rows = torch.empty((T, int(lib.tq_delta_rows_width(c_int(heads), c_int(kv_heads), c_int(dk), c_int(dper)))), dtype=torch.float32, device=xqkv.device)
     check(_LIB, lib.tq_delta_scan_runs(ptr(xqkv), c_int(xqkv.shape[1]), c_int(q_off), c_int(k_off), c_int(v_off), ptr(proj),
-                                       c_int(proj.shape[1]), c_int(b_off), ptr(a_raw), c_int(a_raw.shape[1]), c_int(a_off),
+                                       c_int(proj.shape[1]), c_int(b_off), ptr(a_raw), c_int(a_raw.shape[1]), c_int(a_off), c_int(dper),
                                        ptr(dt_bias), ptr(a_log), ptr(rows), ctypes_ptr(state), c_longlong(state.stride(0)), ptr(y),
                                        c_int(T), c_int(cu_seqlens.shape[0] - 1), c_int(heads), c_int(kv_heads), c_int(dk), c_int(dv),
                                        c_float(unit_eps), c_float(q_scale), ptr(cu_seqlens), ptr(slots), stream()), kernels=2)
     return y
+
+
+def delta_step(xqkv: torch.Tensor, q_off: int, k_off: int, v_off: int, proj: torch.Tensor, b_off: int, a_raw: torch.Tensor,
+               a_off: int, dt_bias: torch.Tensor, a_log: torch.Tensor, gate: torch.Tensor, z_off: int, sigmoid_gate: bool,
+               weight: torch.Tensor, state: torch.Tensor, slots: torch.Tensor, out: torch.Tensor, heads: int, kv_heads: int,
+               dk: int, dv: int, unit_eps: float, q_scale: float, eps: float) -> torch.Tensor:
+    """One token of every sequence through the delta rule in one launch (token t is sequence t, its state the row
+    slots[t]): `delta_scan` and `gated_group_norm(gate_after=True)` over its heads with weight [heads * dv] and the
+    gates' logits gate[:, z_off : z_off + heads * dv].  out [T, heads * dv]."""
+    for t, what in ((xqkv, "q, k and v"), (proj, "the projection"), (a_raw, "the raw decays"), (dt_bias, "the decays' bias"),
+                    (a_log, "the decay rates"), (gate, "the gates"), (state, "the state")):
+        want_f32(t, what)
+    want_int32(slots, "slots")
+    dper = _decays_per_head("delta_step", dt_bias, a_log, heads, dk)
+    T = xqkv.shape[0]
+    if tuple(state.shape[1:]) != (heads, dv, dk) or not state[0].is_contiguous() or out.shape != (T, heads * dv) \
+            or slots.numel() != T or weight.numel() != heads * dv:
+        raise KernelError("delta_step: the state must be [slots, heads, vdim, dim] with dense rows, one slot a token, a weight of heads*dv")
+    lib = load_kernel(_LIB)
+    check(_LIB, lib.tq_delta_step(ptr(xqkv), c_int(xqkv.shape[1]), c_int(q_off), c_int(k_off), c_int(v_off), ptr(proj),
+                                  c_int(proj.shape[1]), c_int(b_off), ptr(a_raw), c_int(a_raw.shape[1]), c_int(a_off), c_int(dper),
+                                  ptr(dt_bias), ptr(a_log), ptr(gate), c_int(gate.shape[1]), c_int(z_off), c_int(1 if sigmoid_gate else 0),
+                                  ptr(weight), c_int(code(weight.dtype)), ctypes_ptr(state), c_longlong(state.stride(0)), ptr(slots),
+                                  ptr(out), c_int(code(out.dtype)), c_int(T), c_int(heads), c_int(kv_heads), c_int(dk), c_int(dv),
+                                  c_float(unit_eps), c_float(q_scale), c_float(eps), stream()))
+    return out
+
+
+# ---- the matrix memory with exponential gates: a sequence's state is S and n as columns [heads, dv + 1, dk] and the
+# running maxima [heads], both views of one row a slot ---------------------------------------------------------------
+
+def _memory_state(what: str, state: torch.Tensor, heads: int, dk: int, dv: int) -> None:
+    want_f32(state, "the state")
+    if tuple(state.shape[1:]) != (heads, dv + 1, dk) or not state[0].is_contiguous():
+        raise KernelError(f"{what}: the state must be [slots, heads, vdim + 1, dim] with dense rows")
+
+
+def memory_gates(proj: torch.Tensor, i_off: int, f_off: int, i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float,
+                 tops_state: torch.Tensor, gates: torch.Tensor, tops: torch.Tensor, heads: int, cu_seqlens: torch.Tensor,
+                 slots: torch.Tensor) -> None:
+    """Log gates of every sequence's run of new tokens: i = cap tanh((raw_i + i_bias) / cap), f = logsigmoid(cap
+    tanh((raw_f + f_bias) / cap)), m = max(f + m_before, i); gates [T, heads, 2] = (f + m_before - m, i - m), tops [T, heads]
+    = m.  tops_state float32 [slots, heads] (rows may be strided): each sequence's m, read and renewed."""
+    for t, what in ((proj, "the projection"), (i_bias, "the input gates' bias"), (f_bias, "the forget gates' bias"),
+                    (tops_state, "the kept maxima"), (gates, "the gates"), (tops, "the maxima")):
+        want_f32(t, what)
+    T = proj.shape[0]
+    if i_bias.numel() != heads or f_bias.numel() != heads or tops_state.shape[1] != heads or tops_state.stride(1) != 1 \
+            or gates.shape != (T, heads, 2) or tops.shape != (T, heads):
+        raise KernelError("memory_gates: biases, kept maxima and outputs must fit the heads")
+    lib = load_kernel(_LIB)
+    check(_LIB, lib.tq_memory_gates(ptr(proj), c_int(proj.shape[1]), c_int(i_off), c_int(f_off), ptr(i_bias), ptr(f_bias), c_float(cap),
+                                    ctypes_ptr(tops_state), c_longlong(tops_state.stride(0)), ptr(gates), ptr(tops),
+                                    c_int(cu_seqlens.shape[0] - 1), c_int(heads), ptr(cu_seqlens), ptr(slots), stream()))
+
+
+def memory_scan(rows: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: torch.Tensor, state: torch.Tensor,
+                y: Optional[torch.Tensor], dots: Optional[torch.Tensor], heads: int, dk: int, dv: int, cu_seqlens: torch.Tensor,
+                slots: torch.Tensor) -> None:
+    """S <- e^gates[..., 0] S + e^gates[..., 1] k v^T, y = S^T q, and with a value of one the same for n, dots = n . q, over every
+    sequence's run.  rows float32 [T, P] with q, k (heads x dk) and v (heads x dv) from the given columns; y [T, heads * dv]
+    and dots [T, heads], or both None: the states are walked on and nothing is written."""
+    want_f32(rows, "q, k and v")
+    want_f32(gates, "the gates")
+    _memory_state("memory_scan", state, heads, dk, dv)
+    for t, what in ((y, "the output"), (dots, "the dot products")):
+        if t is not None:
+            want_f32(t, what)
+    lib = load_kernel(_LIB)
+    check(_LIB, lib.tq_memory_scan(ptr(rows), c_int(rows.shape[1]), c_int(q_off), c_int(k_off), c_int(v_off), ptr(gates), ctypes_ptr(state),
+                                   c_longlong(state.stride(0)), ptr(y), ptr(dots), c_int(cu_seqlens.shape[0] - 1), c_int(heads), c_int(dk),
+                                   c_int(dv), ptr(cu_seqlens), ptr(slots), stream()))
+
+
+def memory_combine(state: torch.Tensor, slots: torch.Tensor, ends: torch.Tensor, starts: torch.Tensor, seq_chunks: torch.Tensor,
+                   cu_chunks: torch.Tensor, gates: torch.Tensor) -> None:
+    """`retention_combine` for chunks that `memory_scan` walked, whose decays are those of their tokens (gates as there)."""
+    for t, what in ((state, "the state"), (ends, "the chunks' states"), (starts, "the chunks' starts"), (gates, "the gates")):
+        want_f32(t, what)
+    for t, what in ((slots, "slots"), (seq_chunks, "the sequences' chunks"), (cu_chunks, "the chunks' tokens")):
+        want_int32(t, what)
+    heads = state.shape[1]
+    if ends.shape != starts.shape or ends.shape[1:] != state.shape[1:] or not (ends.is_contiguous() and starts.is_contiguous()) \
+            or not state[0].is_contiguous() or gates.shape[1:] != (heads, 2) or cu_chunks.numel() != ends.shape[0] + 1:
+        raise KernelError("memory_combine: the chunks' states must be dense and shaped like the kept state's rows")
+    lib = load_kernel(_LIB)
+    check(_LIB, lib.tq_memory_combine(ctypes_ptr(state), c_longlong(state.stride(0)), ptr(slots), ptr(ends), ptr(starts),
+                                      ptr(seq_chunks), ptr(cu_chunks), ptr(gates), c_int(seq_chunks.shape[0] - 1), c_int(heads),
+                                      c_int(state[0, 0].numel()), stream()))
+
+
+def memory_step(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int, i_off: int, f_off: int, i_bias: torch.Tensor,
+                f_bias: torch.Tensor, cap: float, q_scale: float, state: torch.Tensor, tops_state: torch.Tensor,
+                slots: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, heads: int, dk: int, dv: int, floor: float,
+                eps: float) -> torch.Tensor:
+    """One token of every sequence through the memory in one launch (token t is sequence t): `memory_gates`, `memory_scan` and
+    `gated_group_norm(gate_after=True, sigmoid_gate=True, dots=...)` with weight [heads * dv].  out [T, heads * dv]."""
+    for t, what in ((proj, "the projection"), (i_bias, "the input gates' bias"), (f_bias, "the forget gates' bias"),
+                    (tops_state, "the kept maxima")):
+        want_f32(t, what)
+    want_int32(slots, "slots")
+    _memory_state("memory_step", state, heads, dk, dv)
+    T = proj.shape[0]
+    if out.shape != (T, heads * dv) or slots.numel() != T or weight.numel() != heads * dv or i_bias.numel() != heads \
+            or f_bias.numel() != heads or tops_state.shape[1] != heads or tops_state.stride(1) != 1 or tops_state.stride(0) != state.stride(0):
+        raise KernelError("memory_step: one slot a token, a weight and an output of heads*dv, state and maxima in rows of one stride")
+    lib = load_kernel(_LIB)
+    check(_LIB, lib.tq_memory_step(ptr(proj), c_int(proj.shape[1]), c_int(q_off), c_int(k_off), c_int(v_off), c_int(g_off), c_int(i_off),
+                                   c_int(f_off), ptr(i_bias), ptr(f_bias), c_float(cap), c_float(q_scale), ctypes_ptr(state),
+                                   ctypes_ptr(tops_state), c_longlong(state.stride(0)), ptr(slots), ptr(weight), c_int(code(weight.dtype)),
+                                   ptr(out), c_int(code(out.dtype)), c_int(T), c_int(heads), c_int(dk), c_int(dv), c_float(floor),
+                                   c_float(eps), stream()))
+    return out

@@ -6,3 +6,4 @@ from .lumevik import LumevikModel
 from .sisepel import SisepelModel
 from .tasadra import TasadraModel
 from .vukotar import VukotarModel
+from .pamarax import PamaraxModel

@@ -111,6 +111,22 @@ class ExpertRows:
 
 
 @dataclass
+class BranchPair:
+    """What a mixer of two branches leaves to the norm on its output: factors[0] * norm(a) + factors[1] * norm(b), each
+    branch's norm an RMS norm with a weight and `eps` (both weights None: the branches as they are)."""
+    a: torch.Tensor
+    a_weight: Optional[torch.Tensor]
+    b: torch.Tensor
+    b_weight: Optional[torch.Tensor]
+    eps: float
+    factors: Tuple[float, float] = (0.5, 0.5)
+
+    def sum(self) -> torch.Tensor:
+        from ..kernels.elementwise import mean_of_norms
+        return mean_of_norms(self.a, self.a_weight, self.b, self.b_weight, self.eps, torch.empty_like(self.a), self.factors)
+
+
+@dataclass
 class OpenSum:
     """What a block with two sub-layers under one norm leaves to be added to the stream: a_scale * a + b_scale * b, a
     factor per element (float32 [H], or None for one); b is rows like a, ExpertRows, or None.  Only norms that say
@@ -164,9 +180,9 @@ class Norm(Part):
         raise NotImplementedError
 
     def add_normed(self, x: torch.Tensor, y: torch.Tensor, copy: Optional[torch.Tensor] = None, then: Optional["Norm"] = None,
-                   then_dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
-        """x += norm(y) in fp32, for blocks whose norms sit on the sub-layers' outputs; `copy` receives the new x
-        in its own dtype.  then: the norm that reads the new x next; where this norm can take it in the same pass
+                   then_dtype: Optional[torch.dtype] = None, y_bias: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+        """x += norm(y) in fp32 (norm(y + y_bias) with a bias), for blocks whose norms sit on the sub-layers' outputs;
+        `copy` receives the new x in its own dtype.  then: the norm that reads the new x next; where this norm can take it in the same pass
         it returns that norm's output in then_dtype, else None (without `then`: x)."""
         raise NotImplementedError
 

@@ -171,6 +171,10 @@ class BiasedWindowAttentionMixer(Mixer):
         on the same input may compute both projections as one product and hand the rows over (`projected`)."""
         return self.w_qkv
 
+    def take_input_weight(self, w: torch.Tensor) -> None:
+        """The fused input projection as part of a wider one."""
+        self.w_qkv = w
+
     def forward(self, xn: torch.Tensor, ctx: StepContext, cache: LayerCache, projected: Optional[torch.Tensor] = None) -> torch.Tensor:
         """projected: float32 rows that begin with this mixer's [q | k | v] (the rows may be longer); needs the rotating writer."""
         T, act, dev = xn.shape[0], ctx.act_dtype, xn.device

@@ -161,12 +161,13 @@ class SandwichBlock(Block):
         return ["elementwise"] + [k for p in self._direct() for k in p.kernels()]
 
     @staticmethod
-    def _add(norm: Norm, x, y, ctx, copy=None, then: Optional[Norm] = None):
+    def _add(norm: Norm, x, y, ctx, copy=None, then: Optional[Norm] = None, y_bias=None):
         """x += norm(y); returns the norm `then` of the new x where it could be taken in the same pass, else None."""
+        bias = {} if y_bias is None else {"y_bias": y_bias}
         if then is None or not hasattr(norm, "weight"):
-            norm.add_normed(x, y, copy)
+            norm.add_normed(x, y, copy, **bias)
             return None
-        return norm.add_normed(x, y, copy, then=then, then_dtype=ctx.act_dtype)
+        return norm.add_normed(x, y, copy, then=then, then_dtype=ctx.act_dtype, **bias)
 
     def forward(self, x: torch.Tensor, pending: Optional[torch.Tensor], ctx: StepContext,
                 cache: LayerCache) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
@@ -188,19 +189,23 @@ class SandwichBlock(Block):
         then = self.ffn_norm if self.ffn is not None else (out_norm if last else None)
         done = False
         if hasattr(self.mixer, "forward_branches") and hasattr(self.mixer_post, "add_normed_pair"):
-            # a mixer of two normed branches: their norms and mean run inside the sum's pass
+            # a mixer of two branches: their norms and weighted sum run inside the sum's pass
             pair = self.mixer.forward_branches(xn, ctx, cache)
             done, xn = self.mixer_post.add_normed_pair(x, pair, h, then=then, then_dtype=ctx.act_dtype)
             if not done:
-                a, wa, b, wb, eps = pair
-                xn = self._add(self.mixer_post, x, K.mean_of_norms(a, wa, b, wb, eps, torch.empty_like(a)), ctx, copy=h, then=then)
+                xn = self._add(self.mixer_post, x, pair.sum(), ctx, copy=h, then=then)
         else:
             xn = self._add(self.mixer_post, x, self.mixer.forward(xn, ctx, cache), ctx, copy=h, then=then)
         if self.ffn is not None:
             if xn is None:
                 xn = self.ffn_norm.forward(x, ctx.act_dtype)
             h = cast(n_after)
-            xn = self._add(self.ffn_post, x, self.ffn.forward(xn, ctx), ctx, copy=h, then=None if n_after else out_norm)
+            # the bias that ends a feed-forward may be left to the norm on its output (float32)
+            bias = getattr(self.ffn, "down_bias", None)
+            if bias is not None and bias.dtype != torch.float32:
+                bias = bias.float()
+            y = self.ffn.forward(xn, ctx, leave_bias=True) if bias is not None else self.ffn.forward(xn, ctx)
+            xn = self._add(self.ffn_post, x, y, ctx, copy=h, then=None if n_after else out_norm, y_bias=bias)
         for k, part in enumerate(self.after):
             xn = part.apply(x, ctx, cast=h if k == 0 else None, then=out_norm if k == n_after - 1 else None)
         if xn is not None and out_norm is not None:

@@ -51,20 +51,25 @@ register_feed_forward("swiglu", SwiGLUFeedForward)
 class GluFeedForward(FeedForward):
     """down(glu(gate x, up x)) with a gated activation given by its constants (kernels.elementwise.Glu: caps on gate
     and up, the slope inside the sigmoid, an offset on up); the tensors' names are parameters.  Gate and up are
-    one fused product whose float32 result the activation reads."""
+    one fused product whose float32 result the activation reads.  bias: all three products have one (`<name>.b`); a block
+    that adds this part's output to the stream may take the last one into that sum (`forward(..., leave_bias=True)` and
+    `down_bias`)."""
 
     def __init__(self, prefix: str, hidden: int, intermediate: int, glu: K.Glu = K.SILU_GLU, gate_name: str = "gate",
-                 up_name: str = "up", down_name: str = "down"):
+                 up_name: str = "up", down_name: str = "down", bias: bool = False):
         if hidden < 1 or intermediate < 1:
             raise ValueError(f"feed-forward '{prefix}': sizes must be positive, got {hidden}, {intermediate}")
         self.prefix, self.hidden, self.intermediate, self.glu = prefix, int(hidden), int(intermediate), glu
-        self.names = (gate_name, up_name, down_name)
-        self.w_gate_up = self.w_down = None
+        self.names, self.has_bias = (gate_name, up_name, down_name), bool(bias)
+        self.w_gate_up = self.w_down = self.gate_up_bias = self.down_bias = None
 
     def weight_specs(self) -> List[WeightSpec]:
         p, H, I = self.prefix, self.hidden, self.intermediate
-        return [WeightSpec(p + self.names[0], (I, H)), WeightSpec(p + self.names[1], (I, H)),
-                WeightSpec(p + self.names[2], (H, I))]
+        specs = [WeightSpec(p + self.names[0], (I, H)), WeightSpec(p + self.names[1], (I, H)),
+                 WeightSpec(p + self.names[2], (H, I))]
+        if self.has_bias:
+            specs += [WeightSpec(p + n + ".b", (size,)) for n, size in zip(self.names, (I, I, H))]
+        return specs
 
     def bind(self, store: WeightStore) -> None:
         p = self.prefix
@@ -72,6 +77,9 @@ class GluFeedForward(FeedForward):
         dt = torch.float32 if torch.float32 in (g.dtype, u.dtype) else g.dtype
         self.w_gate_up = torch.cat([g.to(dt), u.to(dt)], dim=0).contiguous()
         self.w_down = store.get(p + self.names[2])
+        if self.has_bias:
+            self.gate_up_bias = torch.cat([store.take(p + n + ".b").float() for n in self.names[:2]]).contiguous()
+            self.down_bias = store.take(p + self.names[2] + ".b").float().contiguous()
 
     def kernels(self) -> List[str]:
         return ["elementwise"]
@@ -80,11 +88,14 @@ class GluFeedForward(FeedForward):
         wb = lambda w: 0 if w is None else w.numel() * w.element_size()
         return {"matmul": (wb(self.w_gate_up) + wb(self.w_down), 6.0 * n_tokens * self.hidden * self.intermediate)}
 
-    def forward(self, xn: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+    def forward(self, xn: torch.Tensor, ctx: StepContext, leave_bias: bool = False) -> torch.Tensor:
         gu = linear(xn, self.w_gate_up, out_dtype=torch.float32)
         h = torch.empty((xn.shape[0], self.intermediate), dtype=ctx.act_dtype, device=xn.device)
-        K.glu_mul(gu, h, self.glu)
-        return linear(h, self.w_down, out_dtype=torch.float32)
+        K.glu_mul(gu, h, self.glu, bias=self.gate_up_bias)
+        y = linear(h, self.w_down, out_dtype=torch.float32)
+        if self.down_bias is not None and not leave_bias:
+            K.add_bias(y, self.down_bias)
+        return y
 
 
 register_feed_forward("glu", GluFeedForward)

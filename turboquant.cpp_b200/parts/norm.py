@@ -40,32 +40,32 @@ class RMSNorm(Norm):
         out = torch.empty((x.shape[0], self.size), dtype=out_dtype, device=x.device)
         return K.rmsnorm(x, self.weight, self.eps, out, add=y)
 
-    def add_normed(self, x, y, copy=None, then=None, then_dtype=None):
-        """x += norm(y).  then (an RMSNorm of the same weight dtype): its norm of the new x is taken in the same pass
+    def add_normed(self, x, y, copy=None, then=None, then_dtype=None, y_bias=None):
+        """x += norm(y), or norm(y + y_bias).  then (an RMSNorm of the same weight dtype): its norm of the new x is taken in the same pass
         and returned in then_dtype (None where the two weights' dtypes differ: the caller runs it by itself)."""
         if then is not None and isinstance(then, RMSNorm) and then.weight.dtype == self.weight.dtype and \
                 (copy is None or copy.dtype == then_dtype):
             out = torch.empty((x.shape[0], self.size), dtype=then_dtype, device=x.device)
-            K.add_rmsnorm(x, y, self.weight, self.eps, copy, then.weight, out, then.eps)
+            K.add_rmsnorm(x, y, self.weight, self.eps, copy, then.weight, out, then.eps, y_bias=y_bias)
             return out
-        K.add_rmsnorm(x, y, self.weight, self.eps, copy)
+        K.add_rmsnorm(x, y, self.weight, self.eps, copy, y_bias=y_bias)
         return None if then is not None else x
 
-
     def add_normed_pair(self, x, pair, copy=None, then=None, then_dtype=None):
-        """x += norm(mean of two normed branches); pair = (a, wa, b, wb, eps) as a mixer of two branches leaves them
+        """x += norm(weighted sum of two branches); pair: the BranchPair a mixer of two branches leaves
         (`forward_branches`).  Returns (done, normed): done False where the weights' dtypes differ and nothing was
         computed; normed: the norm `then` of the new x where it was taken along, else None."""
-        a, wa, b, wb, pair_eps = pair
-        if wa.dtype != self.weight.dtype or wb.dtype != self.weight.dtype:
+        if any(w is not None and w.dtype != self.weight.dtype for w in (pair.a_weight, pair.b_weight)):
             return False, None
+        args = (x, pair.a, pair.a_weight, pair.b, pair.b_weight, pair.eps, self.weight, self.eps, copy)
         if then is not None and isinstance(then, RMSNorm) and then.weight.dtype == self.weight.dtype and \
                 (copy is None or copy.dtype == then_dtype):
             out = torch.empty((x.shape[0], self.size), dtype=then_dtype, device=x.device)
-            K.add_rmsnorm_pair(x, a, wa, b, wb, pair_eps, self.weight, self.eps, copy, then.weight, out, then.eps)
+            K.add_rmsnorm_pair(*args, then.weight, out, then.eps, factors=pair.factors)
             return True, out
-        K.add_rmsnorm_pair(x, a, wa, b, wb, pair_eps, self.weight, self.eps, copy)
+        K.add_rmsnorm_pair(*args, factors=pair.factors)
         return True, None
+
 
 register_norm("rmsnorm", RMSNorm)
 

@@ -23,6 +23,7 @@ from ..kernels import ssm as KS
 from ..kernels.linear import linear
 from ..weights.loader import WeightSpec, WeightStore
 from .base import LayerCache, Mixer, StateNeed, StepContext, register_mixer
+from .chunks import cut_runs
 
 
 class RetentionMixer(Mixer):
@@ -43,7 +44,6 @@ class RetentionMixer(Mixer):
         self.k_scale = float(k_scale) if k_scale is not None else float(dim) ** -0.5
         self.qk, self.inner = self.heads * self.dim, self.heads * self.vdim
         self.w_in = self.w_o = self.decay = None
-        self._sm_count: Optional[int] = None
 
     # rows of the fused input projection: [q | k | v | g]
     @property
@@ -81,43 +81,12 @@ class RetentionMixer(Mixer):
         """The fused input projection's weight ([q | k | v | g] rows): see `forward(projected=...)`."""
         return self.w_in
 
-    MIN_CHUNK = 64           # the shortest chunk worth cutting a run into
+    def take_input_weight(self, w: torch.Tensor) -> None:
+        """The fused input projection as part of a wider one."""
+        self.w_in = w
+
     # decode steps with at least this many (sequence, head) pairs take the one-launch form (TQ_RETENTION_STEP_MIN_BLOCKS)
     STEP_MIN_BLOCKS = int(os.environ.get("TQ_RETENTION_STEP_MIN_BLOCKS", "0"))
-
-    def _chunks(self, ctx: StepContext):
-        """None, or how this step's runs are cut into chunks for the recurrence: (token offsets of the chunks
-        [chunks + 1], chunk numbers [chunks], each sequence's chunks [sequences + 1]) on the device.  The recurrence
-        kernel walks a run token by token with a warp per four columns of a head's state; where those warps fill
-        less than half of the GPU and a run is long, cutting the runs fills it, at the price of walking them once
-        more for the states alone (half the work of a walk with outputs).  The plan depends on the step's runs and
-        on heads and vdim only, and is kept for the step's other layers."""
-        lens = list(ctx.host_q_lens)
-        if not lens or len(lens) != ctx.n_seqs or max(lens) < 2 * self.MIN_CHUNK:
-            return None
-        if self._sm_count is None:
-            self._sm_count = torch.cuda.get_device_properties(ctx.device).multi_processor_count
-        cuts = self._sm_count * KS.SCAN_WARPS_PER_SM // KS.scan_warps(len(lens), self.heads, self.vdim)
-        if cuts < 2:
-            return None
-        size = max(self.MIN_CHUNK, -(-max(lens) // cuts))
-        size = -(-size // 16) * 16
-        if max(lens) < 2 * size:
-            return None
-        key = f"retention_chunks_{size}"
-        plan = ctx.carry.get(key) if ctx.carry is not None else None
-        if plan is None:
-            cu, seq_chunks, at = [0], [0], 0
-            for n in lens:
-                for c0 in range(0, n, size):
-                    cu.append(at + min(n, c0 + size))
-                at += n
-                seq_chunks.append(len(cu) - 1)
-            i32 = lambda v: torch.tensor(v, dtype=torch.int32).to(ctx.device, non_blocking=True)
-            plan = (i32(cu), torch.arange(len(cu) - 1, dtype=torch.int32, device=ctx.device), i32(seq_chunks))
-            if ctx.carry is not None:
-                ctx.carry[key] = plan
-        return plan
 
     def forward(self, xn: torch.Tensor, ctx: StepContext, cache: LayerCache, projected: Optional[torch.Tensor] = None,
                 offset: int = 0) -> torch.Tensor:
@@ -139,7 +108,7 @@ class RetentionMixer(Mixer):
                              pe.freq if pe is not None and pe.dims else None, pe.dims if pe is not None else 0,
                              pe is not None and pe.halves, self.k_scale, ctx.positions, self.heads, self.dim, self.vdim)
         y = torch.empty((T, self.inner), dtype=torch.float32, device=dev)
-        plan = self._chunks(ctx)
+        plan = cut_runs(ctx, self.heads, self.vdim)
         if plan is None:
             KS.ssm_scan(xbc, None, 0, None, None, None, S, y, self.heads, self.vdim, self.dim, self.heads, ctx.cu_seqlens,
                         ctx.slots, fixed_decay=self.decay)
