@@ -150,7 +150,7 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 / 64 points and the prefill")
     ap.add_argument("--kernel-table", default="", help="write a per-kernel time table of a few decode steps and of a "
                     "prefill to this file (torch profiler; not part of any timed number)")
-    ap.add_argument("--design", choices=["nuforax", "lumevik", "sisepel", "tasadra", "vukotar"], default="", help="instead of the default workload: prompt "
+    ap.add_argument("--design", choices=["nuforax", "lumevik", "sisepel", "tasadra", "vukotar", "pamarax"], default="", help="instead of the default workload: prompt "
                     "and decode speed of this design at layer sizes of a real model (random weights), beside the closest other "
                     "decoder of equal width, depth and heads")
     ap.add_argument("--sizes", default="w1024,w2048", help="with --design: which of the sizes to run")
@@ -485,6 +485,8 @@ def design_compare(args) -> int:
         return tasadra_compare(args, tq, measure, weights_bytes, pk, rng, prompt, steps, warmup)
     if args.design == "vukotar":
         return vukotar_compare(args, tq, measure, pk, rng, prompt, steps, warmup)
+    if args.design == "pamarax":
+        return pamarax_compare(args, tq, measure, pk, rng, prompt, steps, warmup)
     result = {"metric": "prompt and decode speed, Nuforax beside the dense Qwen2 decoder of equal width", "unit": "tokens/s",
               "n_gpus": 1, "steps": steps, "warmup": warmup, "dtype": "bf16", "data": "synthetic token ids, seeded random weights",
               "peaks": pk, "sizes": {}}
@@ -732,6 +734,65 @@ def vukotar_compare(args, tq, measure, pk, rng, prompt, steps, warmup) -> int:
             if args.kernel_table:
                 kernel_table(tq, model, rng, V, args.batch, args.kernel_table + f".{who}_{name}.txt", prompt=prompt,
                              context=prompt + 128, same_token=False)
+            del model
+            gc.collect()
+            torch.cuda.empty_cache()
+        result["sizes"][name] = entry
+    result["clocks"] = clocks.stop()
+    print(json.dumps(result))
+    return 0
+
+
+def pamarax_config(width, heads, kv_heads, dim, m_heads, m_dim, m_vdim, ff, vocab):
+    """Six layers: matrix memory, attention beside the delta rule, attention, and the three once more; a dense feed-forward
+    on every layer."""
+    memory = {"heads": m_heads, "dim": m_dim, "vdim": m_vdim, "gate_cap": 20.0}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "rot": {"base": 500000.0, "dims": dim // 2}}
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "q_temp": {"coef": 0.2, "every": 1024}}
+    rule = {"heads": heads, "kv_heads": heads, "dim": dim, "vdim": dim, "conv": 4}
+    pair = {"left": left, "right": rule, "left_scale": 0.5, "right_scale": 0.7}
+    mlp = {"kind": "dense", "ff": ff}
+    return {"architecture": "Pamarax", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": width ** 0.5},
+            "layers": [{"type": k, "mixer": m, "mlp": mlp} for k, m in (("mlstm", memory), ("parallel", pair), ("attention", att)) * 2]}
+
+
+PAMARAX_SIZES = {
+    # name: (width, heads, kv heads, head size, matrix memory's (and the sibling's retention) heads, key size, value size,
+    #        feed-forward, vocab)
+    "w1024": (1024, 8, 2, 128, 8, 64, 128, 4096, 32768),
+    "w2048": (2048, 16, 4, 128, 16, 128, 128, 8192, 32768),
+}
+
+
+def pamarax_compare(args, tq, measure, pk, rng, prompt, steps, warmup) -> int:
+    """The Pamarax decoder beside the Sisepel and the Tasadra decoders of the same width, depth, heads, head size and
+    feed-forward size.  Sisepel has norms on both sides of its sub-layers, gated feed-forwards and, on every layer, attention
+    beside a recurrence with a state per head; Tasadra has the other delta rule.  Both see every earlier position here."""
+    import torch
+    result = {"metric": "prompt and decode speed, Pamarax beside the Sisepel and Tasadra decoders of equal sizes", "unit": "tokens/s",
+              "n_gpus": 1, "steps": steps, "warmup": warmup, "dtype": "bf16", "data": "synthetic token ids, seeded random weights",
+              "peaks": pk, "sizes": {}}
+    clocks = ClockSampler()
+    clocks.start()
+    for name in args.sizes.split(","):
+        if name not in PAMARAX_SIZES:
+            print(json.dumps({"error": f"unknown size '{name}'; known: {sorted(PAMARAX_SIZES)}"}))
+            return 2
+        (W, H, G, D, mh, md, mv, ff, V) = PAMARAX_SIZES[name]
+        window = 1 << 20
+        entry = {}
+        for who, cfg in (("pamarax", pamarax_config(W, H, G, D, mh, md, mv, ff, V)),
+                         ("sisepel", sisepel_dense_config(W, 6, H, G, D, window, mh, md, mv, ff, V)),
+                         ("tasadra", tasadra_config(W, H, G, D, D // 2, window, ff, V))):
+            model = tq.random_model(cfg, seed=0, dtype="bfloat16", device="cuda:0")
+            conf = {"width": W, "layers": 6, "heads": H, "kv_heads": G, "head_size": D, "dense_ff": ff}
+            if who != "tasadra":
+                conf.update({"matrix_memory" if who == "pamarax" else "retention": {"heads": mh, "dim": md, "vdim": mv}})
+            if who != "sisepel":
+                conf.update(delta={"heads": H, "dim": D, "vdim": D, "conv": 4})
+            entry[who] = dict(measure(model, V), config=conf)
+            if args.kernel_table:
+                kernel_table(tq, model, rng, V, args.batch, args.kernel_table + f".{who}_{name}.txt", prompt=prompt, context=prompt + 128)
             del model
             gc.collect()
             torch.cuda.empty_cache()

@@ -363,7 +363,7 @@ def memory_step(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: i
     _memory_state("memory_step", state, heads, dk, dv)
     T = proj.shape[0]
     if out.shape != (T, heads * dv) or slots.numel() != T or weight.numel() != heads * dv or i_bias.numel() != heads \
-            or f_bias.numel() != heads or tops_state.shape[1] != heads or tops_state.stride(1) != 1 or tops_state.stride(0) != state.stride(0):
+            or f_bias.numel() != heads or tops_state.shape[1] != heads or tops_state.stride(1) != 1 or (state.shape[0] > 1 and tops_state.stride(0) != state.stride(0)):
         raise KernelError("memory_step: one slot a token, a weight and an output of heads*dv, state and maxima in rows of one stride")
     lib = load_kernel(_LIB)
     check(_LIB, lib.tq_memory_step(ptr(proj), c_int(proj.shape[1]), c_int(q_off), c_int(k_off), c_int(v_off), c_int(g_off), c_int(i_off),
