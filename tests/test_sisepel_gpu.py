@@ -108,8 +108,9 @@ def test_long_prompts_whose_recurrence_runs_in_chunks(folders, name, sizes, dtyp
     """Runs long enough for the retention mixer to cut them into chunks that it scans side by side (whole, and in
     portions that go on from a kept state), beside a short request.  float32: against the plain model.  bfloat16:
     against the same engine with the cutting switched off, position by position (among 700 positions some enlarge a
-    rounding beyond any bound that would still tell a fault; both paths round alike, so they stay together)."""
-    from turboquant_cpp_b200.parts.retention import RetentionMixer
+    rounding beyond any bound that would still tell a fault; both paths round alike, so they stay together where they choose the same
+    experts)."""
+    from turboquant_cpp_b200.parts import retention
     cfg, folder = CONFIGS[name], folders[name]
     toks, other = tokens_for(cfg, sum(sizes), 21), tokens_for(cfg, len(sizes) + 40, 22)
     steps, at = [], 0
@@ -127,21 +128,26 @@ def test_long_prompts_whose_recurrence_runs_in_chunks(folders, name, sizes, dtyp
             eng.release()
 
     cut = []
-    plan = RetentionMixer._chunks
-    monkeypatch.setattr(RetentionMixer, "_chunks", lambda self, ctx: cut.append(plan(self, ctx)) or cut[-1])
+    plan = retention.cut_runs
+    monkeypatch.setattr(retention, "cut_runs", lambda *a: cut.append(plan(*a)) or cut[-1])
     got, routing = run()
     assert any(c is not None for c in cut)                    # the runs were cut
     if dtype == "float32":
         check_against_plain(plain_model(folder), toks, got["p"], routing["p"], dtype, f"{name} long prompt")
         check_against_plain(plain_model(folder), other, got["o"], routing["o"], dtype, f"{name} beside a long prompt")
         return
-    monkeypatch.setattr(RetentionMixer, "_chunks", lambda self, ctx: None)
-    whole, _ = run()
+    monkeypatch.setattr(retention, "cut_runs", lambda *a: None)
+    whole, chosen = run()
     for rid in ("p", "o"):
         ref = np.stack([whole[rid][p] for p in sorted(whole[rid])])
         rows = np.stack([got[rid][p] for p in sorted(whole[rid])])
         d = rows - ref
         e = np.sqrt((d * d).mean(axis=1)) / ref.std()
+        # where a rounding decided between two experts the rows have nothing to do with each other; that is rare
+        same = np.array([all(set(a[p].tolist()) == set(b[p].tolist()) for a, b in zip(routing[rid], chosen[rid]))
+                         for p in sorted(whole[rid])])
+        assert (~same).sum() <= 0.005 * len(same)
+        e = np.where(same, e, 0.0)
         assert e.max() < 2e-2, f"{name} {rid}: position {int(e.argmax())} differs by {e.max():.3e} between the cut and the whole recurrence"
 
 

@@ -137,6 +137,34 @@ __device__ __forceinline__ float tq_rotated(const float* head, int e, int dims, 
     return first ? head[e] * cs - head[partner] * sn : head[e] * cs + head[partner] * sn;
 }
 
+// Two float32 operations in one instruction (sm_100's packed forms of the PTX ISA), each rounded as the single one is.
+typedef unsigned long long tq_f32x2;
+__device__ __forceinline__ tq_f32x2 tq_pack2(float lo, float hi) {
+    tq_f32x2 d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+    return d;
+}
+__device__ __forceinline__ float2 tq_unpack2(tq_f32x2 v) {
+    float2 d;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(d.x), "=f"(d.y) : "l"(v));
+    return d;
+}
+__device__ __forceinline__ tq_f32x2 tq_fma2(tq_f32x2 a, tq_f32x2 b, tq_f32x2 c) {
+    tq_f32x2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ tq_f32x2 tq_mul2(tq_f32x2 a, tq_f32x2 b) {
+    tq_f32x2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ tq_f32x2 tq_add2(tq_f32x2 a, tq_f32x2 b) {
+    tq_f32x2 d;
+    asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+
 __device__ __forceinline__ float tq_warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

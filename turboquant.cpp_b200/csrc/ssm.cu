@@ -25,45 +25,56 @@ TQ_DEFINE_LAST_ERROR
 
 #define CONV_TOKENS 8          // consecutive tokens of a long step per thread: an input is read once, not once per tap
 
-template <typename TW>
-__global__ void conv_silu_kernel(const float* __restrict__ proj, int P, int off, const TW* __restrict__ w,
-                                 const TW* __restrict__ b, const float* __restrict__ kept, long long slot_stride,
-                                 float* __restrict__ out, int T_, int C, int taps, int per_thread, const int* __restrict__ seq_of_token,
-                                 const int* __restrict__ cu_seqlens, const int* __restrict__ slots, int n_seqs) {
+// PER tokens and TAPS taps at most per thread (fewer taps: the others are zero)
+template <typename TW, int PER, int TAPS>
+__global__ void __launch_bounds__(128)
+conv_silu_kernel(const float* __restrict__ proj, int P, int off, const TW* __restrict__ w,
+                 const TW* __restrict__ b, const float* __restrict__ kept, long long slot_stride,
+                 float* __restrict__ out, int T_, int C, int taps, const int* __restrict__ seq_of_token,
+                 const int* __restrict__ cu_seqlens, const int* __restrict__ slots, int n_seqs) {
     tq_grid_wait();                    // everything below may read what the previous kernel wrote
     tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
-    const int tb = blockIdx.x * per_thread, c = blockIdx.y * blockDim.x + threadIdx.x;
+    const int tb = blockIdx.x * PER, c = blockIdx.y * blockDim.x + threadIdx.x;
     if (c >= C) return;
-    // win[SSM_MAX_TAPS - 1 - k] is the input k positions back; wr the tap that meets it (0 beyond the taps)
-    float win[SSM_MAX_TAPS], wr[SSM_MAX_TAPS];
+    const int n = min(PER, T_ - tb);
+    const float* in = proj + (size_t)tb * P + off + c;
+    float x[PER];                      // the thread's inputs, all on their way together
 #pragma unroll
-    for (int k = 0; k < SSM_MAX_TAPS; ++k) {
-        win[SSM_MAX_TAPS - 1 - k] = 0.f;
-        wr[SSM_MAX_TAPS - 1 - k] = k < taps ? tq_to_float(w[(size_t)c * taps + taps - 1 - k]) : 0.f;
+    for (int k = 0; k < PER; ++k) x[k] = k < n ? in[(size_t)k * P] : 0.f;
+    // win[TAPS - 1 - k] is the input k positions back; wr the tap that meets it (0 beyond the taps)
+    float win[TAPS], wr[TAPS];
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k) {
+        win[TAPS - 1 - k] = 0.f;
+        wr[TAPS - 1 - k] = k < taps ? tq_to_float(w[(size_t)c * taps + taps - 1 - k]) : 0.f;
     }
     const float bias = b ? tq_to_float(b[c]) : 0.f;
-    const int t_end = min(T_, tb + per_thread);
-    for (int t = tb; t < t_end; ++t) {
-        const int s = TQ_CHECKED(seq_of_token[t], n_seqs, TQ_IDX_SEQUENCE);
-        const int i = t - cu_seqlens[s];             // place in the sequence's run of new tokens
-        if (t == tb || i == 0) {                     // the thread's first token, or a new sequence: the inputs before it
-            const float* old = kept + (size_t)slots[s] * slot_stride;      // [taps-1][C]: inputs of the positions just before the run
+    int s = TQ_CHECKED(seq_of_token[tb], n_seqs, TQ_IDX_SEQUENCE), end = tb;      // `end`: where the sequence's run ends
 #pragma unroll
-            for (int k = 1; k < SSM_MAX_TAPS; ++k) {
-                if (k < taps) {
-                    const int src = i - k;
-                    win[SSM_MAX_TAPS - 1 - k] = src >= 0 ? proj[(size_t)(t - k) * P + off + c]
-                                                         : old[(size_t)(taps - 1 + src) * C + c];
+    for (int j = 0; j < PER; ++j) {
+        const int t = tb + j;
+        if (j < n) {
+            if (j == 0 || t == end) {                    // the thread's first token, or a new sequence: the inputs before it
+                if (j > 0) s = TQ_CHECKED(seq_of_token[t], n_seqs, TQ_IDX_SEQUENCE);
+                end = cu_seqlens[s + 1];
+                const int i = t - cu_seqlens[s];         // place in the sequence's run of new tokens
+                const float* old = kept + (size_t)slots[s] * slot_stride;      // [taps-1][C]: inputs of the positions just before the run
+#pragma unroll
+                for (int k = 1; k < TAPS; ++k) {
+                    if (k < taps) {
+                        const int src = i - k;
+                        win[TAPS - 1 - k] = src >= 0 ? in[((long long)j - k) * P] : old[(size_t)(taps - 1 + src) * C + c];
+                    }
                 }
             }
+            win[TAPS - 1] = x[j];
+            float acc = bias;
+#pragma unroll
+            for (int k = 0; k < TAPS; ++k) acc += wr[k] * win[k];
+            out[(size_t)t * C + c] = acc / (1.0f + expf(-acc));
+#pragma unroll
+            for (int k = 0; k < TAPS - 1; ++k) win[k] = win[k + 1];
         }
-        win[SSM_MAX_TAPS - 1] = proj[(size_t)t * P + off + c];
-        float acc = bias;
-#pragma unroll
-        for (int k = 0; k < SSM_MAX_TAPS; ++k) acc += wr[k] * win[k];
-        out[(size_t)t * C + c] = acc / (1.0f + expf(-acc));
-#pragma unroll
-        for (int k = 0; k < SSM_MAX_TAPS - 1; ++k) win[k] = win[k + 1];
     }
 }
 
@@ -139,9 +150,14 @@ TQ_EXPORT int tq_conv_silu(const float* proj, int P, int off, const void* w, con
     const int per_thread = T_ >= 256 ? CONV_TOKENS : 1;        // short steps keep a thread per token and channel
     dim3 grid((T_ + per_thread - 1) / per_thread, (C + threads - 1) / threads);
     TQ_REQUIRE(grid.y <= 65535, "conv_silu: %d channels exceed the grid limit", C);
-    TQ_DISPATCH(w_dtype, TW,
-        (tq_launch(grid, threads, 0, stream)(conv_silu_kernel<TW>, proj, P, off, (const TW*)w, (const TW*)b,
-                                             (const float*)kept, slot_stride, out, T_, C, taps, per_thread, seq_of_token, cu_seqlens, slots, n_seqs)));
+#define CONV_LAUNCH(PER, TAPS)                                                                                          \
+    TQ_DISPATCH(w_dtype, TW,                                                                                            \
+        (tq_launch(grid, threads, 0, stream)(conv_silu_kernel<TW, PER, TAPS>, proj, P, off, (const TW*)w, (const TW*)b,  \
+                                             (const float*)kept, slot_stride, out, T_, C, taps, seq_of_token, cu_seqlens, slots, n_seqs)))
+    if (per_thread == 1) CONV_LAUNCH(1, SSM_MAX_TAPS);
+    else if (taps <= 4) CONV_LAUNCH(CONV_TOKENS, 4);
+    else CONV_LAUNCH(CONV_TOKENS, SSM_MAX_TAPS);
+#undef CONV_LAUNCH
     TQ_CHECK_LAUNCH("conv_silu");
     if (taps > 1) {
         dim3 ugrid(n_seqs, (C + threads - 1) / threads);
@@ -154,9 +170,9 @@ TQ_EXPORT int tq_conv_silu(const float* proj, int P, int off, const void* w, con
 // ---------------------------------------------------------------------------------------
 // ssm_scan: grid (sequences, heads, ceil(vdim / SSM_COLS)), SSM_COLS / SSM_CPW warps per block.  A warp owns
 // SSM_CPW neighbouring columns of the head's state (kept column by column, [vdim][N], so the lanes' loads and
-// stores are neighbours in memory): lane l keeps rows l, l+32, ... (RPL of them) of each column in registers for
+// stores are neighbours in memory): lane l keeps RPL rows of each column, in neighbouring pairs, in registers for
 // the whole run, so a step reads its B and C values once for the warp's columns and does three float32 operations
-// per element of the state (the product B x, the decayed sum, the sum for y).  The sums of y over the lanes are
+// per element of the state (the product B x, the decayed sum, the sum for y), two elements an instruction.  The sums of y over the lanes are
 // not taken step by step: 32 / SSM_CPW steps leave 32 partial sums per lane, which five rounds of exchanges (31
 // shuffles) turn into one whole sum per lane, so the chain of dependent shuffles is paid once per group of steps
 // and the state's updates run on meanwhile; a whole group is straight-line code.  No barrier between steps.  The
@@ -171,7 +187,8 @@ TQ_EXPORT int tq_conv_silu(const float* proj, int P, int off, const void* w, con
 //   x_cols                columns of x; a state column from x_cols on (at most one) has x = 1: its state is the decayed sum
 //                         of B alone, and its read-out goes to `ones_out` [T, heads] instead of y [T, heads x x_cols]
 //   log_gates             per token and head the logarithms of the decay and of the step size, [T, heads] pairs (the
-//                         per-head constants and the raw step sizes are then not read)
+//                         per-head constants and the raw step sizes are then not read); a walk without outputs then leaves
+//                         every run's decay, the product of its tokens', in ones_out [sequences, heads]
 struct SsmRows {
     int x_off, b_off, c_off, x_cols;
     const float2* log_gates;
@@ -212,14 +229,19 @@ ssm_scan_kernel(const float* __restrict__ xbc, int C, const float* __restrict__ 
     const float A = fixed ? 0.f : -expf(tq_to_float(a_log[h])), bias = fixed ? 0.f : tq_to_float(dt_bias[h]);
     const float D = fixed ? 0.f : tq_to_float(d_skip[h]), decay_h = fixed_decay != nullptr ? fixed_decay[h] : 0.f;
     float* Sg = state + (size_t)slots[s] * slot_stride + ((size_t)h * N) * vdim;
-    float S[RPL][SSM_CPW];
+    // a lane's rows come in neighbouring pairs, 2 lane + 64 r and the one behind it, so that two rows' operations are one
+    // packed instruction (with up to 32 rows: one row a lane, two columns' operations packed)
+    constexpr bool ROWS2 = RPL > 1;
+    constexpr int SR = ROWS2 ? RPL / 2 : 1, SC = ROWS2 ? SSM_CPW : SSM_CPW / 2;
+    tq_f32x2 S[SR][SC];
+    auto cell = [&](int row, int col) -> float* { return row < N && vw + col < vdim ? Sg + (size_t)(vw + col) * N + row : nullptr; };
+    auto get = [](const float* p) { return p ? *p : 0.f; };
 #pragma unroll
-    for (int r = 0; r < RPL; ++r) {
+    for (int r = 0; r < SR; ++r) {
 #pragma unroll
-        for (int c = 0; c < SSM_CPW; ++c) {
-            const int row = lane + 32 * r;
-            S[r][c] = (row < N && vw + c < vdim) ? Sg[(size_t)(vw + c) * N + row] : 0.f;
-        }
+        for (int c = 0; c < SC; ++c)
+            S[r][c] = ROWS2 ? tq_pack2(get(cell(2 * lane + 64 * r, c)), get(cell(2 * lane + 64 * r + 1, c)))
+                            : tq_pack2(get(cell(lane, 2 * c)), get(cell(lane, 2 * c + 1)));
     }
     constexpr int LPT = TC * NP / NT;                    // B and C values per thread and chunk
     constexpr int XPT = TC * SSM_COLS / NT;              // x values per thread and chunk
@@ -245,6 +267,7 @@ ssm_scan_kernel(const float* __restrict__ xbc, int C, const float* __restrict__ 
         if (tid < tc && gates) pgate = gates[(size_t)(first + t0 + tid) * heads + h];
         if (tid < tc && !fixed) praw = proj[(size_t)(first + t0 + tid) * P + dt_off + h];
     };
+    float log_decay = 0.f;                   // without outputs: the first warp's share of the run's log decay
     if (n > 0) fetch(0);
     for (int t0 = 0; t0 < n; t0 += TC) {
         const int tc = min(TC, n - t0);
@@ -259,6 +282,7 @@ ssm_scan_kernel(const float* __restrict__ xbc, int C, const float* __restrict__ 
             const float raw = praw + bias;
             const float dt = fixed ? 1.0f : (raw > 20.f ? raw : log1pf(expf(raw)));
             dts[tid] = gates ? expf(pgate.y) : dt;
+            if constexpr (!OUT) log_decay += pgate.x;
             dec[tid] = gates ? expf(pgate.x) : (fixed ? decay_h : expf(A * dt));
         }
         __syncthreads();
@@ -274,22 +298,39 @@ ssm_scan_kernel(const float* __restrict__ xbc, int C, const float* __restrict__ 
 #pragma unroll
                     for (int c = 0; c < SSM_CPW; ++c) v[j * SSM_CPW + c] = 0.f;
                     if (decltype(full)::value || tt < tc) {          // the same for the whole block
-                        float xv[SSM_CPW];
-                        if constexpr (SSM_CPW == 4) {
-                            const float4 x4 = *reinterpret_cast<const float4*>(xs + tt * SSM_COLS + warp * SSM_CPW);
-                            xv[0] = x4.x; xv[1] = x4.y; xv[2] = x4.z; xv[3] = x4.w;
+                        const float* xp = xs + tt * SSM_COLS + warp * SSM_CPW;
+                        const tq_f32x2 a2 = tq_pack2(dec[tt], dec[tt]), dt2 = tq_pack2(dts[tt], dts[tt]);
+                        auto pair = [](const float* p) { return *reinterpret_cast<const tq_f32x2*>(p); };
+                        tq_f32x2 o[SC];
+                        if constexpr (ROWS2) {
+                            tq_f32x2 x2[SC];
+#pragma unroll
+                            for (int c = 0; c < SC; ++c) x2[c] = tq_pack2(xp[c], xp[c]);
+#pragma unroll
+                            for (int r = 0; r < SR; ++r) {
+                                const tq_f32x2 b2 = tq_mul2(pair(Bs + tt * NP + 2 * lane + 64 * r), dt2);
+                                const tq_f32x2 c2 = pair(Cs + tt * NP + 2 * lane + 64 * r);
+#pragma unroll
+                                for (int c = 0; c < SC; ++c) {
+                                    S[r][c] = tq_fma2(a2, S[r][c], tq_mul2(b2, x2[c]));
+                                    if constexpr (OUT) o[c] = r == 0 ? tq_mul2(S[r][c], c2) : tq_fma2(S[r][c], c2, o[c]);
+                                }
+                            }
+                            if constexpr (OUT) {
+#pragma unroll
+                                for (int c = 0; c < SC; ++c) { const float2 u = tq_unpack2(o[c]); v[j * SSM_CPW + c] = u.x + u.y; }
+                            }
                         } else {
-                            const float2 x2 = *reinterpret_cast<const float2*>(xs + tt * SSM_COLS + warp * SSM_CPW);
-                            xv[0] = x2.x; xv[1] = x2.y;
-                        }
-                        const float a = dec[tt], dt = dts[tt];
+                            const float bv = Bs[tt * NP + lane], cv = Cs[tt * NP + lane];
+                            const tq_f32x2 b2 = tq_mul2(tq_pack2(bv, bv), dt2), c2 = tq_pack2(cv, cv);
 #pragma unroll
-                        for (int r = 0; r < RPL; ++r) {
-                            const float bv = Bs[tt * NP + lane + 32 * r] * dt, cv = Cs[tt * NP + lane + 32 * r];
-#pragma unroll
-                            for (int c = 0; c < SSM_CPW; ++c) {
-                                S[r][c] = a * S[r][c] + bv * xv[c];
-                                if constexpr (OUT) v[j * SSM_CPW + c] += S[r][c] * cv;
+                            for (int c = 0; c < SC; ++c) {
+                                S[0][c] = tq_fma2(a2, S[0][c], tq_mul2(b2, pair(xp + 2 * c)));
+                                if constexpr (OUT) {
+                                    const float2 u = tq_unpack2(tq_mul2(S[0][c], c2));
+                                    v[j * SSM_CPW + 2 * c] = u.x;
+                                    v[j * SSM_CPW + 2 * c + 1] = u.y;
+                                }
                             }
                         }
                     }
@@ -318,12 +359,20 @@ ssm_scan_kernel(const float* __restrict__ xbc, int C, const float* __restrict__ 
         }
         __syncthreads();
     }
+    if constexpr (!OUT) {
+        if (gates && blockIdx.z == 0 && warp == 0) {                   // a chunk's steps are the first warp's lanes (TC <= 32)
+            log_decay = tq_warp_sum(log_decay);
+            if (lane == 0) rows.ones_out[(size_t)s * heads + h] = expf(log_decay);
+        }
+    }
+    auto put = [](float* p, float value) { if (p) *p = value; };
 #pragma unroll
-    for (int r = 0; r < RPL; ++r) {
+    for (int r = 0; r < SR; ++r) {
 #pragma unroll
-        for (int c = 0; c < SSM_CPW; ++c) {
-            const int row = lane + 32 * r;
-            if (row < N && vw + c < vdim) Sg[(size_t)(vw + c) * N + row] = S[r][c];
+        for (int c = 0; c < SC; ++c) {
+            const float2 u = tq_unpack2(S[r][c]);
+            put(ROWS2 ? cell(2 * lane + 64 * r, c) : cell(lane, 2 * c), u.x);
+            put(ROWS2 ? cell(2 * lane + 64 * r + 1, c) : cell(lane, 2 * c + 1), u.y);
         }
     }
 }
@@ -732,7 +781,7 @@ TQ_EXPORT int tq_retention_step(const float* proj, int P, int q_off, int k_off, 
 //   memory_gates    both logarithms of every token and head, and m, of a run of tokens: m is a scan over the tokens with
 //                   the operation (F1, M1) then (F2, M2) = (F1 + F2, max(M1 + F2, M2))
 //   memory_scan     the recurrence (a launcher of ssm_scan_kernel; y and n . q without their denominators)
-//   memory_combine  retention_combine for decays that differ from token to token
+//   memory_combine  retention_combine with a decay per chunk
 //   memory_step     a step of single tokens in one launch: gates, the state's update and read-out, denominator, RMS norm,
 //                   weight and the sigmoid of the output gate
 // The denominators, norms and output gates of a run are gated_group_norm's (`part`).
@@ -762,11 +811,21 @@ memory_gates_kernel(const float* __restrict__ proj, int P, int i_off, int f_off,
     const float bi = i_bias[h], bf = f_bias[h];
     float before = *kept;              // m ahead of the tile's first token
     int buf = 0;
+    float raw_i = 0.f, raw_f = 0.f;
+    auto ask = [&](int at) {
+        if (at < n) {
+            const float* row = proj + ((size_t)first + at) * P;
+            raw_i = row[i_off + h];
+            raw_f = row[f_off + h];
+        }
+    };
+    ask(tid);
     for (int base = 0; base < n; base += MEM_GATE_THREADS, buf ^= 1) {
         const bool live = base + tid < n;
         const size_t t = (size_t)first + base + tid;
         MemGate g = {-INFINITY, 0.f};
-        if (live) g = memory_gate(proj[t * P + i_off + h] + bi, proj[t * P + f_off + h] + bf, cap);
+        if (live) g = memory_gate(raw_i + bi, raw_f + bf, cap);
+        ask(base + MEM_GATE_THREADS + tid);            // the next tile's, on their way while this one is scanned
         float F = g.f, M = g.i;
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
@@ -806,60 +865,43 @@ TQ_EXPORT int tq_memory_gates(const float* proj, int P, int i_off, int f_off, co
 }
 
 // rows fp32 [T, C] with q, k (heads x dk) and v (heads x dv); state rows of [heads][dv + 1][dk]; y fp32 [T, heads * dv] and dots
-// fp32 [T, heads] (n . q), or both null: the states are walked on and nothing is written.
+// fp32 [T, heads] (n . q); or y null: the states are walked on, nothing is written, and dots [sequences, heads] receives every
+// run's decay (the product of its tokens').
 TQ_EXPORT int tq_memory_scan(const float* rows, int C, int q_off, int k_off, int v_off, const void* gates, float* state,
                              long long slot_stride, float* y, float* dots, int n_seqs, int heads, int dk, int dv,
                              const int* cu_seqlens, const int* slots, cudaStream_t stream) {
     if (n_seqs == 0) return 0;
-    TQ_REQUIRE(gates != nullptr && (y == nullptr) == (dots == nullptr), "memory_scan: gates, and both outputs or neither%s", "");
+    TQ_REQUIRE(gates != nullptr && dots != nullptr, "memory_scan: gates and somewhere for the dot products or decays%s", "");
     const SsmRows in = {v_off, k_off, q_off, dv, (const float2*)gates, dots};
     return ssm_scan_launch(rows, C, nullptr, 0, 0, nullptr, nullptr, nullptr, TQ_F32, state, slot_stride, y, n_seqs, heads, dv + 1, dk,
                            heads, cu_seqlens, slots, nullptr, in, stream);
 }
 
-// As retention_combine, a chunk's decay being e to the sum of its tokens' log decays.  Grid (elements of a head / 256, heads,
-// sequences): the block adds up its head's log decays of the sequence's chunks first (a warp per chunk), MEM_CHUNKS at a time.
-#define MEM_CHUNKS 64
+// As retention_combine, with a decay per chunk and head (decays [chunks, heads]).  Grid (elements / 256, sequences).
 __global__ void __launch_bounds__(256)
 memory_combine_kernel(float* __restrict__ state, long long slot_stride, const int* __restrict__ slots,
                       const float* __restrict__ ends, float* __restrict__ starts, const int* __restrict__ seq_chunks,
-                      const int* __restrict__ cu_chunks, const float2* __restrict__ gates, int heads, int per_head) {
+                      const float* __restrict__ decays, int heads, int per_head) {
     tq_grid_wait();                    // everything below may read what the previous kernel wrote
     tq_grid_launch_dependents();       // the next kernel's CTAs may move in as SMs free up
-    __shared__ float s_decay[MEM_CHUNKS];
-    const int h = blockIdx.y, s = blockIdx.z, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int e = blockIdx.x * blockDim.x + threadIdx.x;
-    const bool live = e < per_head;
-    const int c_end = seq_chunks[s + 1];
-    float* cell = state + (size_t)slots[s] * slot_stride + (size_t)h * per_head + (live ? e : 0);
-    float S = live ? *cell : 0.f;
-    for (int c0 = seq_chunks[s]; c0 < c_end; c0 += MEM_CHUNKS) {
-        const int nc = min(MEM_CHUNKS, c_end - c0);
-        for (int c = warp; c < nc; c += blockDim.x >> 5) {
-            float sum = 0.f;
-            for (int t = cu_chunks[c0 + c] + lane; t < cu_chunks[c0 + c + 1]; t += 32) sum += gates[(size_t)t * heads + h].x;
-            sum = tq_warp_sum(sum);
-            if (lane == 0) s_decay[c] = expf(sum);
-        }
-        __syncthreads();
-        if (live)
-            for (int c = 0; c < nc; ++c) {
-                const size_t at = ((size_t)(c0 + c) * heads + h) * per_head + e;
-                starts[at] = S;
-                S = s_decay[c] * S + ends[at];
-            }
-        __syncthreads();
+    const int n_elems = heads * per_head, e = blockIdx.x * blockDim.x + threadIdx.x, s = blockIdx.y;
+    if (e >= n_elems) return;
+    const int h = e / per_head;
+    float* cell = state + (size_t)slots[s] * slot_stride + e;
+    float S = *cell;
+    for (int c = seq_chunks[s]; c < seq_chunks[s + 1]; ++c) {
+        starts[(size_t)c * n_elems + e] = S;
+        S = decays[(size_t)c * heads + h] * S + ends[(size_t)c * n_elems + e];
     }
-    if (live) *cell = S;
+    *cell = S;
 }
 
 TQ_EXPORT int tq_memory_combine(float* state, long long slot_stride, const int* slots, const float* ends, float* starts,
-                                const int* seq_chunks, const int* cu_chunks, const void* gates, int n_seqs, int heads,
-                                int per_head, cudaStream_t stream) {
+                                const int* seq_chunks, const float* decays, int n_seqs, int heads, int per_head, cudaStream_t stream) {
     if (n_seqs == 0) return 0;
-    TQ_REQUIRE(heads >= 1 && heads <= 65535 && per_head >= 1 && n_seqs <= 65535, "memory_combine: %d heads of %d in %d sequences", heads, per_head, n_seqs);
-    tq_launch(dim3((per_head + 255) / 256, heads, n_seqs), 256, 0, stream)(memory_combine_kernel, state, slot_stride, slots, ends, starts,
-        seq_chunks, cu_chunks, (const float2*)gates, heads, per_head);
+    TQ_REQUIRE(heads >= 1 && per_head >= 1 && n_seqs <= 65535, "memory_combine: %d heads of %d in %d sequences", heads, per_head, n_seqs);
+    tq_launch(dim3((heads * per_head + 255) / 256, n_seqs), 256, 0, stream)(memory_combine_kernel, state, slot_stride, slots, ends, starts,
+        seq_chunks, decays, heads, per_head);
     TQ_CHECK_LAUNCH("memory_combine");
     return 0;
 }
@@ -1124,12 +1166,13 @@ TQ_EXPORT int tq_delta_scan(const float* xqkv, int C, int q_off, int k_off, int 
 //   delta_prepare: what the recurrence reads, for all tokens side by side: per token a row of `R` floats
 //                  [k: G x dk unit vectors | q: G x dk unit vectors times q_scale | g: H x dper decays | k.q: G | beta: H]
 //                  (R rounded up to a multiple of four).  A warp per (token, query/key head) and per (token, head).
-//   delta_scan_rows: the recurrence over those rows.  Same grid and ownership of the state as delta_scan; a chunk's
-//                  rows come through cp.async into one of two buffers in shared memory while the chunk before is
-//                  computed.  Per token both read-outs are taken from the decayed state BEFORE the write,
+//   delta_scan_rows: the recurrence over those rows.  Same grid and split of the columns as delta_scan (four warps; a lane's
+//                  rows in neighbouring pairs, two to an instruction); four more warps bring a chunk's rows through cp.async
+//                  into one of two buffers in shared memory while the chunk before is walked.  Per token both read-outs are taken from the decayed state BEFORE the write,
 //                  pred = (gS)^T k and r = (gS)^T q, their two chains of shuffles side by side, and the output is
 //                  o = r + (k.q) u: the same sum as (gS + k u^T)^T q, with one round of shuffles on the path from a
-//                  token's state to the next token's instead of two.  With one decay per head (HEAD_DECAY) the sums are
+//                  token's state to the next token's instead of two.  Only pred is summed over the lanes token by
+//                  token; r's partial sums of eight tokens are added up together.  With one decay per head (HEAD_DECAY) the sums are
 //                  taken of the undecayed state and multiplied afterwards, off the state's own path.
 // ---------------------------------------------------------------------------------------
 __global__ void __launch_bounds__(128)
@@ -1181,7 +1224,7 @@ __device__ __forceinline__ void delta_copy16(float* smem_dst, const float* src) 
 }
 
 template <int RPL, bool HEAD_DECAY>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256, RPL <= 16 ? 2 : 1)
 delta_scan_rows_kernel(const float* __restrict__ rows, int R, const float* __restrict__ xqkv, int C, int v_off,
                        float* __restrict__ state, long long slot_stride, float* __restrict__ y, int heads, int kv_heads,
                        int dk, int dv, int tc, int vec, const int* __restrict__ cu_seqlens, const int* __restrict__ slots) {
@@ -1193,19 +1236,21 @@ delta_scan_rows_kernel(const float* __restrict__ rows, int R, const float* __res
     const int per_buf = tc * (VECS * DKP + DELTA_COLS + 4);    // k, q, g rows, values, k.q, beta (and a head's g, and one unused) per token
     const int s = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * DELTA_COLS;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, sub = lane & 7;
-    const int lc = warp * 4 + (lane >> 3), col = c0 + lc;
-    const bool live = col < dv;
+    const bool walks = warp < 4;         // four warps walk the recurrence, four bring the next chunk's rows meanwhile
+    const int lc = (warp & 3) * 4 + (lane >> 3), col = c0 + lc, ft = threadIdx.x - 128;
+    const bool live = walks && col < dv;
     const int g = h / (heads / kv_heads);
     const int t0 = cu_seqlens[s], n = cu_seqlens[s + 1] - t0;
     const int g_at = 2 * kv_heads * dk, kq_at = g_at + heads * (HEAD_DECAY ? 1 : dk), b_at = kq_at + kv_heads;
     for (int i = threadIdx.x; i < 2 * per_buf; i += blockDim.x) delta_rows_smem[i] = 0.f;      // rows beyond dk stay zero
     __syncthreads();
     float* Sp = state + (size_t)slots[s] * slot_stride + ((size_t)h * dv + (live ? col : 0)) * dk;
-    float S[RPL];
+    constexpr int NP = RPL / 2;          // a lane's rows come in neighbouring pairs: 2 sub + 16 r and the one behind it
+    tq_f32x2 S[NP];
 #pragma unroll
-    for (int r = 0; r < RPL; ++r) {
-        const int row = sub + 8 * r;
-        S[r] = live && row < dk ? Sp[row] : 0.f;
+    for (int r = 0; r < NP; ++r) {
+        const int row = 2 * sub + 16 * r;
+        S[r] = tq_pack2(live && row < dk ? Sp[row] : 0.f, live && row + 1 < dk ? Sp[row + 1] : 0.f);
     }
     auto fetch = [&](int base, int buf) {
         float* b = delta_rows_smem + (size_t)buf * per_buf;
@@ -1213,7 +1258,7 @@ delta_scan_rows_kernel(const float* __restrict__ rows, int R, const float* __res
         const int nt = min(tc, n - base);
         if (vec) {
             const int q4 = dk >> 2;
-            for (int i = threadIdx.x; i < nt * q4; i += blockDim.x) {
+            for (int i = ft; i < nt * q4; i += 128) {
                 const int tk = i / q4, e = (i - tk * q4) * 4;
                 const float* src = rows + ((size_t)t0 + base + tk) * R;
                 delta_copy16(bk + tk * DKP + e, src + (size_t)g * dk + e);
@@ -1221,7 +1266,7 @@ delta_scan_rows_kernel(const float* __restrict__ rows, int R, const float* __res
                 if constexpr (!HEAD_DECAY) delta_copy16(bg + tk * DKP + e, src + g_at + (size_t)h * dk + e);
             }
         } else {
-            for (int i = threadIdx.x; i < nt * dk; i += blockDim.x) {
+            for (int i = ft; i < nt * dk; i += 128) {
                 const int tk = i / dk, e = i - tk * dk;
                 const float* src = rows + ((size_t)t0 + base + tk) * R;
                 delta_copy4(bk + tk * DKP + e, src + (size_t)g * dk + e);
@@ -1230,7 +1275,7 @@ delta_scan_rows_kernel(const float* __restrict__ rows, int R, const float* __res
             }
         }
         constexpr int ONES = HEAD_DECAY ? 3 : 2;                 // single numbers per token
-        for (int i = threadIdx.x; i < nt * (DELTA_COLS + ONES); i += blockDim.x) {
+        for (int i = ft; i < nt * (DELTA_COLS + ONES); i += 128) {
             const int tk = i / (DELTA_COLS + ONES), e = i - tk * (DELTA_COLS + ONES);
             const size_t t = (size_t)t0 + base + tk;
             if (e < DELTA_COLS) {
@@ -1243,61 +1288,101 @@ delta_scan_rows_kernel(const float* __restrict__ rows, int R, const float* __res
                 delta_copy4(bs + tk * 4 + 2, rows + t * R + g_at + h);
             }
         }
-        asm volatile("cp.async.commit_group;" ::: "memory");
+        asm volatile("cp.async.wait_all;" ::: "memory");
     };
-    if (n > 0) fetch(0, 0);
+    if (n > 0 && !walks) fetch(0, 0);
     int buf = 0;
     for (int base = 0; base < n; base += tc, buf ^= 1) {
+        __syncthreads();                 // this chunk's rows are there, and the other buffer has been walked
+        if (!walks) {
+            if (base + tc < n) fetch(base + tc, buf ^ 1);
+            continue;
+        }
         const int nt = min(tc, n - base);
-        if (base + tc < n) {
-            fetch(base + tc, buf ^ 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();
         const float* b = delta_rows_smem + (size_t)buf * per_buf;
-        const float* bk = b + sub; const float* bq = bk + tc * DKP; const float* bg = bq + tc * DKP;
+        const float* bk = b + 2 * sub; const float* bq = bk + tc * DKP; const float* bg = bq + tc * DKP;
         const float* bv = b + VECS * tc * DKP; const float* bs = bv + tc * DELTA_COLS;
-        for (int i = 0; i < nt; ++i) {
-            float kreg[RPL];
-            float p0 = 0.f, p1 = 0.f, r0 = 0.f, r1 = 0.f;
+        for (int i8 = 0; i8 < nt; i8 += 8) {
+            float part[8], ku = 0.f;             // the read-outs' partial sums of eight tokens; (k.q) u of token i8 + sub
+            auto tokens = [&](auto full) {
+                // a whole group runs as straight-line code; a token's vectors are in registers before the token ahead is done
+                tq_f32x2 kc[NP], qc[NP], gc[HEAD_DECAY ? 1 : NP];
+                float vc;
+                float4 oc;                       // k.q, beta, a head's g
+                auto pair = [](const float* p) { return *reinterpret_cast<const tq_f32x2*>(p); };
+                auto load = [&](int i) {
 #pragma unroll
-            for (int r = 0; r < RPL; r += 2) {
-                kreg[r] = bk[i * DKP + 8 * r];
-                kreg[r + 1] = bk[i * DKP + 8 * (r + 1)];
-                if constexpr (!HEAD_DECAY) {
-                    S[r] *= bg[i * DKP + 8 * r];
-                    S[r + 1] *= bg[i * DKP + 8 * (r + 1)];
+                    for (int r = 0; r < NP; ++r) {
+                        kc[r] = pair(bk + i * DKP + 16 * r);
+                        qc[r] = pair(bq + i * DKP + 16 * r);
+                        if constexpr (!HEAD_DECAY) gc[r] = pair(bg + i * DKP + 16 * r);
+                    }
+                    oc = *reinterpret_cast<const float4*>(bs + i * 4);
+                    vc = bv[i * DELTA_COLS + lc];
+                };
+                auto sum4 = [](const tq_f32x2* p) {
+                    const float2 a = tq_unpack2(tq_add2(tq_add2(p[0], p[1]), tq_add2(p[2], p[3])));
+                    return a.x + a.y;
+                };
+                load(i8);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    part[j] = 0.f;
+                    if (decltype(full)::value || i8 + j < nt) {      // the same for the whole block
+                        tq_f32x2 p[4] = {0, 0, 0, 0}, o[4] = {0, 0, 0, 0}, k[NP];
+#pragma unroll
+                        for (int r = 0; r < NP; ++r) {
+                            k[r] = kc[r];
+                            if constexpr (!HEAD_DECAY) S[r] = tq_mul2(S[r], gc[r]);
+                            p[r & 3] = r < 4 ? tq_mul2(S[r], k[r]) : tq_fma2(S[r], k[r], p[r & 3]);
+                        }
+                        float pred = sum4(p);
+                        if constexpr (HEAD_DECAY) pred *= oc.z;
+                        pred += __shfl_xor_sync(0xffffffffu, pred, 1);
+#pragma unroll
+                        for (int r = 0; r < NP; ++r) o[r & 3] = r < 4 ? tq_mul2(S[r], qc[r]) : tq_fma2(S[r], qc[r], o[r & 3]);
+                        part[j] = sum4(o);
+                        if constexpr (HEAD_DECAY) {
+                            part[j] *= oc.z;
+                            const tq_f32x2 g2 = tq_pack2(oc.z, oc.z);
+#pragma unroll
+                            for (int r = 0; r < NP; ++r) S[r] = tq_mul2(S[r], g2);
+                        }
+                        const float kq = oc.x, beta = oc.y, v = vc;
+                        if (j < 7) load(i8 + j + 1);       // a partial group reads rows of the buffer that hold older tokens
+                        pred += __shfl_xor_sync(0xffffffffu, pred, 2);
+                        pred += __shfl_xor_sync(0xffffffffu, pred, 4);
+                        const float u = beta * (v - pred);
+                        const tq_f32x2 u2 = tq_pack2(u, u);
+#pragma unroll
+                        for (int r = 0; r < NP; ++r) S[r] = tq_fma2(k[r], u2, S[r]);
+                        if (sub == j) ku = kq * u;
+                    }
                 }
-                p0 += S[r] * kreg[r];
-                p1 += S[r + 1] * kreg[r + 1];
-                r0 += S[r] * bq[i * DKP + 8 * r];
-                r1 += S[r + 1] * bq[i * DKP + 8 * (r + 1)];
-            }
-            float pred = p0 + p1, rd = r0 + r1;
-            pred += __shfl_xor_sync(0xffffffffu, pred, 1);
-            rd += __shfl_xor_sync(0xffffffffu, rd, 1);
-            pred += __shfl_xor_sync(0xffffffffu, pred, 2);
-            rd += __shfl_xor_sync(0xffffffffu, rd, 2);
-            pred += __shfl_xor_sync(0xffffffffu, pred, 4);
-            rd += __shfl_xor_sync(0xffffffffu, rd, 4);
-            if constexpr (HEAD_DECAY) { pred *= bs[i * 4 + 2]; rd *= bs[i * 4 + 2]; }
-            const float u = bs[i * 4 + 1] * (bv[i * DELTA_COLS + lc] - pred);
+            };
+            if (i8 + 8 <= nt) tokens(std::true_type{});
+            else tokens(std::false_type{});
+            // eight sums over a column's eight lanes: every round a lane keeps the half of its values that its bit names
+            // and gets the other lane's share of it, so that lane `sub` ends up with the whole sum of token i8 + sub
 #pragma unroll
-            for (int r = 0; r < RPL; ++r) {
-                if constexpr (HEAD_DECAY) S[r] = bs[i * 4 + 2] * S[r] + kreg[r] * u;
-                else S[r] += kreg[r] * u;
+            for (int half = 4; half >= 1; half >>= 1) {
+                const bool up = sub & half;
+#pragma unroll
+                for (int k = 0; k < half; ++k) {
+                    const float keep = up ? part[k + half] : part[k], send = up ? part[k] : part[k + half];
+                    part[k] = keep + __shfl_xor_sync(0xffffffffu, send, half);
+                }
             }
-            if (sub == 0 && live) y[((size_t)t0 + base + i) * heads * dv + (size_t)h * dv + col] = rd + bs[i * 4] * u;
+            if (live && i8 + sub < nt) y[((size_t)t0 + base + i8 + sub) * heads * dv + (size_t)h * dv + col] = part[0] + ku;
         }
-        __syncthreads();                 // the buffer is free for the chunk after the next
     }
     if (live) {
 #pragma unroll
-        for (int r = 0; r < RPL; ++r) {
-            const int row = sub + 8 * r;
-            if (row < dk) Sp[row] = S[r];
+        for (int r = 0; r < NP; ++r) {
+            const int row = 2 * sub + 16 * r;
+            const float2 v = tq_unpack2(S[r]);
+            if (row < dk) Sp[row] = v.x;
+            if (row + 1 < dk) Sp[row + 1] = v.y;
         }
     }
 }
@@ -1344,7 +1429,7 @@ TQ_EXPORT int tq_delta_scan_runs(const float* xqkv, int C, int q_off, int k_off,
             cudaFuncSetAttribute(delta_scan_rows_kernel<RP, HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024); \
             roomy = true;                                                                                              \
         }                                                                                                              \
-        tq_launch(grid, 128, smem, stream, 1, few_blocks ? false : true)(delta_scan_rows_kernel<RP, HD>, (const float*)rows, R, xqkv, C, \
+        tq_launch(grid, 256, smem, stream, 1, few_blocks ? false : true)(delta_scan_rows_kernel<RP, HD>, (const float*)rows, R, xqkv, C, \
             v_off, state, slot_stride, y, heads, kv_heads, dk, dv, tc, vec, cu_seqlens, slots);                         \
     } while (0)
     if (head_decay) {

@@ -316,17 +316,19 @@ def memory_gates(proj: torch.Tensor, i_off: int, f_off: int, i_bias: torch.Tenso
 
 
 def memory_scan(rows: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: torch.Tensor, state: torch.Tensor,
-                y: Optional[torch.Tensor], dots: Optional[torch.Tensor], heads: int, dk: int, dv: int, cu_seqlens: torch.Tensor,
+                y: Optional[torch.Tensor], dots: torch.Tensor, heads: int, dk: int, dv: int, cu_seqlens: torch.Tensor,
                 slots: torch.Tensor) -> None:
     """S <- e^gates[..., 0] S + e^gates[..., 1] k v^T, y = S^T q, and with a value of one the same for n, dots = n . q, over every
     sequence's run.  rows float32 [T, P] with q, k (heads x dk) and v (heads x dv) from the given columns; y [T, heads * dv]
-    and dots [T, heads], or both None: the states are walked on and nothing is written."""
+    and dots [T, heads]; or y None: the states are walked on, and dots [sequences, heads] receives every run's decay."""
     want_f32(rows, "q, k and v")
     want_f32(gates, "the gates")
     _memory_state("memory_scan", state, heads, dk, dv)
-    for t, what in ((y, "the output"), (dots, "the dot products")):
-        if t is not None:
-            want_f32(t, what)
+    want_f32(dots, "the dot products or decays")
+    if y is not None:
+        want_f32(y, "the output")
+    if dots.numel() != heads * (rows.shape[0] if y is not None else cu_seqlens.shape[0] - 1):
+        raise KernelError("memory_scan: a dot product per token and head, or a decay per run and head")
     lib = load_kernel(_LIB)
     check(_LIB, lib.tq_memory_scan(ptr(rows), c_int(rows.shape[1]), c_int(q_off), c_int(k_off), c_int(v_off), ptr(gates), ctypes_ptr(state),
                                    c_longlong(state.stride(0)), ptr(y), ptr(dots), c_int(cu_seqlens.shape[0] - 1), c_int(heads), c_int(dk),
@@ -334,19 +336,19 @@ def memory_scan(rows: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: t
 
 
 def memory_combine(state: torch.Tensor, slots: torch.Tensor, ends: torch.Tensor, starts: torch.Tensor, seq_chunks: torch.Tensor,
-                   cu_chunks: torch.Tensor, gates: torch.Tensor) -> None:
-    """`retention_combine` for chunks that `memory_scan` walked, whose decays are those of their tokens (gates as there)."""
-    for t, what in ((state, "the state"), (ends, "the chunks' states"), (starts, "the chunks' starts"), (gates, "the gates")):
+                   decays: torch.Tensor) -> None:
+    """`retention_combine` for chunks that `memory_scan` walked without outputs; decays [chunks, heads] as it leaves them."""
+    for t, what in ((state, "the state"), (ends, "the chunks' states"), (starts, "the chunks' starts"), (decays, "the decays")):
         want_f32(t, what)
-    for t, what in ((slots, "slots"), (seq_chunks, "the sequences' chunks"), (cu_chunks, "the chunks' tokens")):
+    for t, what in ((slots, "slots"), (seq_chunks, "the sequences' chunks")):
         want_int32(t, what)
     heads = state.shape[1]
     if ends.shape != starts.shape or ends.shape[1:] != state.shape[1:] or not (ends.is_contiguous() and starts.is_contiguous()) \
-            or not state[0].is_contiguous() or gates.shape[1:] != (heads, 2) or cu_chunks.numel() != ends.shape[0] + 1:
+            or not state[0].is_contiguous() or decays.numel() != ends.shape[0] * heads:
         raise KernelError("memory_combine: the chunks' states must be dense and shaped like the kept state's rows")
     lib = load_kernel(_LIB)
     check(_LIB, lib.tq_memory_combine(ctypes_ptr(state), c_longlong(state.stride(0)), ptr(slots), ptr(ends), ptr(starts),
-                                      ptr(seq_chunks), ptr(cu_chunks), ptr(gates), c_int(seq_chunks.shape[0] - 1), c_int(heads),
+                                      ptr(seq_chunks), ptr(decays), c_int(seq_chunks.shape[0] - 1), c_int(heads),
                                       c_int(state[0, 0].numel()), stream()))
 
 

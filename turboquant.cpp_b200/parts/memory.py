@@ -105,8 +105,9 @@ class MatrixMemoryMixer(Mixer):
                 cu_chunks, chunk_ids, seq_chunks = plan
                 ends = torch.zeros((chunk_ids.shape[0], H, dv + 1, dk), dtype=torch.float32, device=dev)
                 starts = torch.empty_like(ends)
-                scan(ends, None, None, cu_chunks, chunk_ids)
-                KS.memory_combine(S, ctx.slots, ends, starts, seq_chunks, cu_chunks, gates)
+                decays = f32(chunk_ids.shape[0], H)
+                scan(ends, None, decays, cu_chunks, chunk_ids)
+                KS.memory_combine(S, ctx.slots, ends, starts, seq_chunks, decays)
                 scan(starts, y, dots, cu_chunks, chunk_ids)
             KS.gated_group_norm(y, proj, z, self.w_norm, H, self.eps, o, gate_after=True, sigmoid_gate=True, dots=dots, tops=m,
                                 dot_scale=dk ** -0.5, floor=DENOMINATOR_FLOOR)
