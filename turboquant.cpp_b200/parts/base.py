@@ -202,6 +202,8 @@ class PositionEncoding(Part):
 
 
 class Mixer(Part):
+    runs_alone = False            # whether runs of many tokens go through a long kernel of few blocks that wants the GPU to itself
+
     def cache_need(self) -> Optional[KVNeed]:
         return None
 

@@ -6,13 +6,13 @@ sub-layer's output as `pending` and hands its own feed-forward output on the sam
 sum is one fp32 pass together with the next norm's statistics."""
 from __future__ import annotations
 
-import os
 from typing import List, Optional, Tuple
 
 import torch
 
 from ..kernels import elementwise as K
 from ..weights.loader import WeightSpec, WeightStore
+from . import side
 from .base import Block, FeedForward, KVNeed, LayerCache, Mixer, Norm, OpenSum, StateNeed, StepContext
 
 
@@ -224,8 +224,7 @@ class ParallelBlock(Block):
     next (an OpenSum; a routed feed-forward's weighted sum over its experts joins it), which must be of a kind that
     takes one; else the block adds it up itself."""
 
-    _side_streams = {}
-    SIDE_BY_SIDE = os.environ.get("TQ_NO_SIDE_BY_SIDE", "") in ("", "0")
+    SIDE_BY_SIDE = side.ENABLED
     # prompts whose stream holds fewer elements run on one stream: launches, not the GPU, bound such a step, and the fork
     # and join are launches too (measured on B200, ms of a 2,048-token prompt through four layers on one stream / two:
     # width 1,024: 1.60 / 1.68, width 2,048: 2.57 / 2.43); decode steps are replayed as graphs
@@ -266,13 +265,6 @@ class ParallelBlock(Block):
     def kernels(self) -> List[str]:
         return ["elementwise"] + [k for p in self.parts() for k in p.kernels()]
 
-    @classmethod
-    def _side_stream(cls, device):
-        key = torch.device(device).index
-        if key not in cls._side_streams:
-            cls._side_streams[key] = torch.cuda.Stream(device=device)
-        return cls._side_streams[key]
-
     def forward(self, x: torch.Tensor, pending, ctx: StepContext, cache: LayerCache):
         if isinstance(pending, OpenSum) and not self.norm.adds_open_sums:
             K.branches_dyt(x, **pending.operands())
@@ -284,15 +276,11 @@ class ParallelBlock(Block):
         f = None
         run_ffn = lambda: self.ffn.forward(h, ctx, leave_rows=True) if hasattr(self.ffn, "n_experts") else self.ffn.forward(h, ctx)
         if self.ffn is not None and self.SIDE_BY_SIDE and (ctx.max_q_len == 1 or x.numel() >= self.SIDE_MIN_ELEMENTS):
-            # what the feed-forward allocates on the second stream is read by the sum on this one and not used again
-            # before the second stream has waited for this one, at the next layer's fork: no block of memory is
-            # handed out while the other stream still reads it
-            main, side = torch.cuda.current_stream(), self._side_stream(x.device)
-            side.wait_stream(main)
-            with torch.cuda.stream(side):
+            other = side.fork(x.device)
+            with torch.cuda.stream(other):
                 f = run_ffn()
             y = self.mixer.forward(h, ctx, cache)
-            main.wait_stream(side)
+            side.join(other)
         else:
             y = self.mixer.forward(h, ctx, cache)
             f = run_ffn() if self.ffn is not None else None

@@ -35,6 +35,7 @@ UNIT_EPS = 1e-6          # inside the root of the unit vectors of q and k
 
 
 class ChannelDeltaMixer(Mixer):
+    runs_alone = True
     RUNS_MIN = 16             # steps whose longest run of new tokens is at least this take the two-launch form
 
     def __init__(self, prefix: str, hidden: int, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, eps: float,
@@ -135,6 +136,7 @@ register_mixer("channel_delta", ChannelDeltaMixer)
 class HeadDeltaMixer(Mixer):
     """The delta rule with one decay per head (see the module's header)."""
 
+    runs_alone = True
     RUNS_MIN = ChannelDeltaMixer.RUNS_MIN
 
     def __init__(self, prefix: str, hidden: int, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, eps: float):

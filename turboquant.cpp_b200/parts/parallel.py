@@ -17,10 +17,18 @@ import torch
 
 from ..kernels.linear import linear
 from ..weights.loader import WeightSpec, WeightStore
+from . import side
 from .base import BranchPair, KVNeed, LayerCache, Mixer, StateNeed, StepContext, register_mixer
 
 
 class ParallelMixer(Mixer):
+    # The branches run on two streams: neither waits for the other.  Prompts stay on one where launches, not the GPU, bound
+    # the step (a smaller stream), and where a branch wants the GPU to itself.  Measured on B200, one stream / two: decoding
+    # with a delta rule beside attention 0.588 / 0.566 ms (batch 8, width 2,048), with retention 0.692 / 0.674 ms; a prompt
+    # with retention 5.79 / 5.26 ms, with a delta rule 4.33 / 4.49 ms.
+    SIDE_BY_SIDE = side.ENABLED
+    SIDE_MIN_ELEMENTS = 3 << 20
+
     def __init__(self, left: Mixer, right: Mixer, hidden: int, eps: float, left_norm: Optional[str] = None,
                  right_norm: Optional[str] = None, factors: Tuple[float, float] = (0.5, 0.5)):
         """left_norm, right_norm: the names of the two norms' weights (both None: no norms)."""
@@ -73,13 +81,20 @@ class ParallelMixer(Mixer):
     def forward_branches(self, xn: torch.Tensor, ctx: StepContext, cache: LayerCache) -> BranchPair:
         """The two branches' outputs before their norms, for a block whose norm on the mixer's output takes the
         branches' norms and their weighted sum in its own pass."""
+        left_in, right_in = {}, {}
         if self.w_in is not None:
             proj = linear(xn, self.w_in, out_dtype=torch.float32)
-            a = self.left.forward(xn, ctx, cache, projected=proj)
-            b = self.right.forward(xn, ctx, cache, projected=proj, offset=self.left.input_weight().shape[0])
+            left_in, right_in = {"projected": proj}, {"projected": proj, "offset": self.left.input_weight().shape[0]}
+        runs_apart = xn.numel() >= self.SIDE_MIN_ELEMENTS and not (self.left.runs_alone or self.right.runs_alone)
+        if self.SIDE_BY_SIDE and (ctx.max_q_len == 1 or runs_apart):
+            other = side.fork(xn.device)
+            with torch.cuda.stream(other):
+                b = self.right.forward(xn, ctx, cache, **right_in)
+            a = self.left.forward(xn, ctx, cache, **left_in)
+            side.join(other)
         else:
-            a = self.left.forward(xn, ctx, cache)
-            b = self.right.forward(xn, ctx, cache)
+            a = self.left.forward(xn, ctx, cache, **left_in)
+            b = self.right.forward(xn, ctx, cache, **right_in)
         return BranchPair(a, self.w_left, b, self.w_right, self.eps, self.factors)
 
     def forward(self, xn: torch.Tensor, ctx: StepContext, cache: LayerCache) -> torch.Tensor:
