@@ -12,6 +12,10 @@ where pre and post are RMS norms whose stored weight is the distance from one.  
 exponential gates; softmax attention whose values are its unnormed, unrotated keys, with a norm over the whole query and
 key rows, and a gate per element; and two branches side by side, softmax attention with one more in the softmax's
 denominator and a temperature on the queries, and a delta rule with one decay per head.
+
+`store` (identity by default) is applied wherever an implementation with 16-bit activations keeps one: what the norms hand
+to the products, attention's queries, keys, values and sums, what enters a mixer's last product, and the feed-forward's
+inner activations.  With `to_bfloat16` the model is what such an implementation computes, up to its float32 sums.
 """
 import json
 import math
@@ -74,6 +78,16 @@ def unit_rms(v, eps):
     return v / np.sqrt(np.mean(v * v, axis=-1, keepdims=True) + eps)
 
 
+def keep(v):
+    return v
+
+
+def to_bfloat16(v):
+    """To the nearest bfloat16, ties to even."""
+    u = np.ascontiguousarray(v, dtype=np.float32).view(np.uint32).astype(np.uint64)
+    return (((u + 0x7FFF + ((u >> 16) & 1)) >> 16) << 16).astype(np.uint32).view(np.float32).astype(F)
+
+
 def around_one(v, w, eps):
     """An RMS norm whose stored weight is the distance from one."""
     return unit_rms(v, eps) * (1.0 + w)
@@ -105,7 +119,7 @@ def memory_gates(h, w, p, cap):
     return capped("i"), log_sigmoid(capped("f"))
 
 
-def memory_mixer(h, w, p, m, eps):
+def memory_mixer(h, w, p, m, eps, store=keep):
     T = h.shape[0]
     H, dim, vdim = m["heads"], m["dim"], m["vdim"]
     q = (h @ w[p + "q"].T).reshape(T, H, dim) * dim ** -0.5
@@ -116,7 +130,7 @@ def memory_mixer(h, w, p, m, eps):
     for a in range(H):
         o[:, a], _ = memory_recurrence(q[:, a], k[:, a], v[:, a], gi[:, a], gf[:, a])
     o = unit_rms(o, eps).reshape(T, H * vdim) * w[p + "norm"]
-    return (o * sigmoid(h @ w[p + "g"].T)) @ w[p + "o"].T
+    return store(o * sigmoid(h @ w[p + "g"].T)) @ w[p + "o"].T
 
 
 # ---- softmax attention --------------------------------------------------------------------------------------------
@@ -150,7 +164,7 @@ def attend(q, k, v, scale, extra=0.0):
     return out
 
 
-def shared_value_attention(h, w, p, m, eps):
+def shared_value_attention(h, w, p, m, eps, store=keep):
     T = h.shape[0]
     H, G, dim = m["heads"], m["kv_heads"], m["dim"]
     pos = np.arange(T)
@@ -161,15 +175,15 @@ def shared_value_attention(h, w, p, m, eps):
     rot = m.get("rot")
     if rot and rot["dims"]:
         q, k = (rotate_halves(u, pos, rot["dims"], rot["base"]) for u in (q, k))
-    o = attend(q, k, v, m["scale"]).reshape(T, H * dim)
-    return (o * sigmoid(h @ w[p + "g"].T)) @ w[p + "o"].T
+    o = store(attend(store(q), store(k), store(v), m["scale"])).reshape(T, H * dim)
+    return store(o * sigmoid(h @ w[p + "g"].T)) @ w[p + "o"].T
 
 
 def query_temperature(positions, coef, every):
     return 1.0 + coef * np.log(np.floor((positions + 1) / every) + 1.0)
 
 
-def sink_attention(h, w, p, m, eps):
+def sink_attention(h, w, p, m, eps, store=keep):
     T = h.shape[0]
     H, G, dim, vdim = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
     q = unit_rms((h @ w[p + "q"].T).reshape(T, H, dim), eps) * w[p + "q.norm"]
@@ -178,7 +192,8 @@ def sink_attention(h, w, p, m, eps):
     temp = m.get("q_temp")
     if temp:
         q = q * query_temperature(np.arange(T), temp["coef"], temp["every"])[:, None, None]
-    return attend(q, k, v, m["scale"], extra=1.0).reshape(T, H * vdim) @ w[p + "o"].T
+    o = attend(store(q), store(k), store(v), m["scale"], extra=1.0)
+    return store(o.reshape(T, H * vdim)) @ w[p + "o"].T
 
 
 # ---- delta rule with one decay per head -----------------------------------------------------------------------------
@@ -211,7 +226,7 @@ def gated_delta_rule(q, k, v, beta, decay, S=None):
     return out, S
 
 
-def delta_mixer(h, w, p, m, eps):
+def delta_mixer(h, w, p, m, eps, store=keep):
     T = h.shape[0]
     H, G, dim, vdim = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
     q, k, v = (silu(short_convolution(h @ w[p + n].T, w[p + n + ".conv"])) for n in ("q", "k", "v"))
@@ -225,42 +240,42 @@ def delta_mixer(h, w, p, m, eps):
         g = a // (H // G)
         o[:, a], _ = gated_delta_rule(q[:, g], k[:, g], v[:, a], beta[:, a], decay[:, a])
     o = unit_rms(o, eps) * w[p + "norm"] * silu(h @ w[p + "g"].T).reshape(T, H, vdim)
-    return o.reshape(T, H * vdim) @ w[p + "o"].T
+    return store(o.reshape(T, H * vdim)) @ w[p + "o"].T
 
 
-def parallel_mixer(h, w, p, m, eps):
-    return (m["left_scale"] * sink_attention(h, w, p + "left.", m["left"], eps) +
-            m["right_scale"] * delta_mixer(h, w, p + "right.", m["right"], eps))
+def parallel_mixer(h, w, p, m, eps, store=keep):
+    return (m["left_scale"] * sink_attention(h, w, p + "left.", m["left"], eps, store) +
+            m["right_scale"] * delta_mixer(h, w, p + "right.", m["right"], eps, store))
 
 
 MIXERS = {"mlstm": memory_mixer, "attention": shared_value_attention, "parallel": parallel_mixer}
 
 
 # ---- feed-forward and model -----------------------------------------------------------------------------------------
-def feed_forward(h, w, p):
+def feed_forward(h, w, p, store=keep):
     lin = lambda u, n: u @ w[p + n].T + w[p + n + ".b"]
-    return lin(silu(lin(h, "gate")) * lin(h, "up"), "down")
+    return lin(store(silu(lin(h, "gate")) * lin(h, "up")), "down")
 
 
-def forward(cfg, w, tokens, streams=None):
+def forward(cfg, w, tokens, streams=None, store=keep):
     """Logits [T, vocab] of a whole sequence; `streams` (a list) receives the stream after every layer."""
     eps = cfg["norm"]["eps"]
     x = w["embed"][np.asarray(tokens)] * cfg["embedding"]["scale"]
     for i, layer in enumerate(cfg["layers"]):
         p = f"l{i}."
-        y = MIXERS[layer["type"]](around_one(x, w[p + "norm1"], eps), w, p + "mix.", layer["mixer"], eps)
+        y = MIXERS[layer["type"]](store(around_one(x, w[p + "norm1"], eps)), w, p + "mix.", layer["mixer"], eps, store)
         x = x + around_one(y, w[p + "norm1b"], eps)
         if layer.get("mlp") is not None:
-            y = feed_forward(around_one(x, w[p + "norm2"], eps), w, p + "mlp.")
+            y = feed_forward(store(around_one(x, w[p + "norm2"], eps)), w, p + "mlp.", store)
             x = x + around_one(y, w[p + "norm2b"], eps)
         if streams is not None:
             streams.append(x.copy())
-    return around_one(x, w["final.norm"], eps) @ w["head"].T
+    return store(around_one(x, w["final.norm"], eps)) @ w["head"].T
 
 
 class PlainPamarax:
     def __init__(self, folder):
         self.cfg, self.weights = load(folder)
 
-    def forward(self, tokens, streams=None):
-        return forward(self.cfg, self.weights, tokens, streams)
+    def forward(self, tokens, streams=None, store=keep):
+        return forward(self.cfg, self.weights, tokens, streams, store)
