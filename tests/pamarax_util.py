@@ -4,8 +4,9 @@ import numpy as np
 from nuforax_util import run_steps, spread_error, write_folder      # noqa: F401  (file writing, schedules)
 
 # float32: sums of a few thousand terms in another order than float64.  bfloat16, against the plain model rounded where the
-# engine rounds: single activations fall on the other side of a rounding, and norms on the sub-layers' outputs enlarge that.
-TOL = {"float32": (1e-5, 1e-4), "bfloat16": (3e-2, 0.15)}      # (nine positions in ten, every position)
+# engine rounds: single activations fall on the other side of a rounding, the tensor-core attention kernels also round the
+# softmax's weights, and norms on the sub-layers' outputs enlarge both at single positions.
+TOL = {"float32": (1e-5, 1e-4), "bfloat16": (2e-2, 0.3)}      # (nine positions in ten, every position)
 
 
 def assert_close(got_rows, ref, dtype, what):
