@@ -906,10 +906,21 @@ TQ_EXPORT int tq_memory_combine(float* state, long long slot_stride, const int* 
     return 0;
 }
 
+// How many warps share a head's columns, four at a time, in a step of single tokens: up to sixteen, or eight where the launch
+// has blocks enough to fill the GPU several times over (smaller blocks, whose phases then overlap with their neighbours').
+// TQ_STEP_WARPS=N: at most N.
+static int step_warps(long long blocks, int groups) {
+    static const int most = [] { const char* e = getenv("TQ_STEP_WARPS"); return e && atoi(e) > 0 ? atoi(e) : 0; }();
+    const int cap = most ? most : (blocks >= 400 ? 8 : 16);
+    int w = 1;
+    while (2 * w <= cap && 2 * w <= groups && w < 16) w *= 2;
+    return w;
+}
+
 // Grid (token, head): up to sixteen warps take four columns of S at a time, one more warp the column n.
 #define MEM_STEP_COLS 4
 template <int RPL, typename TW, typename TO>
-__global__ void __launch_bounds__(544)
+__global__ void __launch_bounds__(544, RPL <= 4 ? 2 : 1)
 memory_step_kernel(const float* __restrict__ proj, int P, int q_off, int k_off, int v_off, int g_off, int i_off, int f_off,
                    const float* __restrict__ i_bias, const float* __restrict__ f_bias, float cap, float q_scale,
                    float* __restrict__ state, float* __restrict__ top_state, long long slot_stride,
@@ -927,6 +938,18 @@ memory_step_kernel(const float* __restrict__ proj, int P, int q_off, int k_off, 
     const float* vr = row + v_off + (size_t)h * dv;
     float* S = state + (size_t)slots[t] * slot_stride + (size_t)h * (dv + 1) * dk;
     float* top = top_state + (size_t)slots[t] * slot_stride + h;
+    // a group of columns' state is asked for as early as possible: the first before anything else, the others before the
+    // sums over the group ahead
+    float sv[RPL][MEM_STEP_COLS];
+    auto load = [&](int c0) {
+#pragma unroll
+        for (int i = 0; i < RPL; ++i) {
+            const int r = lane + 32 * i;
+#pragma unroll
+            for (int j = 0; j < MEM_STEP_COLS; ++j) sv[i][j] = (r < dk && c0 + j < dv) ? S[(size_t)(c0 + j) * dk + r] : 0.f;
+        }
+    };
+    if (warp < n_warps) load(warp * MEM_STEP_COLS);
     const MemGate g = memory_gate(row[i_off + h] + i_bias[h], row[f_off + h] + f_bias[h], cap);
     const float m_old = *top, m = fmaxf(g.f + m_old, g.i);
     const float keep = expf(g.f + m_old - m), take = expf(g.i - m);
@@ -954,13 +977,6 @@ memory_step_kernel(const float* __restrict__ proj, int P, int q_off, int k_off, 
     } else {
         for (int c0 = warp * MEM_STEP_COLS; c0 < dv; c0 += n_warps * MEM_STEP_COLS) {
             float vc[MEM_STEP_COLS], acc[MEM_STEP_COLS];
-            float sv[RPL][MEM_STEP_COLS];               // all of the columns' state in registers first
-#pragma unroll
-            for (int i = 0; i < RPL; ++i) {
-                const int r = lane + 32 * i;
-#pragma unroll
-                for (int j = 0; j < MEM_STEP_COLS; ++j) sv[i][j] = (r < dk && c0 + j < dv) ? S[(size_t)(c0 + j) * dk + r] : 0.f;
-            }
 #pragma unroll
             for (int j = 0; j < MEM_STEP_COLS; ++j) {
                 vc[j] = c0 + j < dv ? vr[c0 + j] : 0.f;
@@ -978,6 +994,7 @@ memory_step_kernel(const float* __restrict__ proj, int P, int q_off, int k_off, 
                     }
                 }
             }
+            load(c0 + n_warps * MEM_STEP_COLS);        // beyond dv: zeros, nothing is read
 #pragma unroll
             for (int j = 0; j < MEM_STEP_COLS; ++j) acc[j] = tq_warp_sum(acc[j]);
             if (lane == 0) {
@@ -1011,7 +1028,7 @@ TQ_EXPORT int tq_memory_step(const float* proj, int P, int q_off, int k_off, int
                k_off + heads * dk <= P && v_off + heads * dv <= P && g_off + heads * dv <= P && i_off + heads <= P && f_off + heads <= P,
                "memory_step: the heads lie outside the projection's rows of %d", P);
     const int groups = (dv + MEM_STEP_COLS - 1) / MEM_STEP_COLS;
-    const int threads = 32 * (groups >= 16 ? 16 : (groups >= 8 ? 8 : (groups >= 4 ? 4 : (groups >= 2 ? 2 : 1)))) + 32;
+    const int threads = 32 * step_warps((long long)T_ * heads, groups) + 32;
 #define MEM_STEP_LAUNCH(R)                                                                                              \
     TQ_DISPATCH(w_dtype, TW, TQ_DISPATCH(out_dtype, TO,                                                                 \
         (tq_launch(dim3(T_, heads), threads, (size_t)dv * sizeof(float), stream)(memory_step_kernel<R, TW, TO>, proj, P, q_off, k_off, v_off, \
@@ -1452,7 +1469,7 @@ TQ_EXPORT int tq_delta_scan_runs(const float* xqkv, int C, int q_off, int k_off,
 // ---------------------------------------------------------------------------------------
 #define DELTA_STEP_COLS 4
 template <int RPL, typename TW, typename TO>
-__global__ void __launch_bounds__(512)
+__global__ void __launch_bounds__(512, RPL <= 4 ? 2 : 1)
 delta_step_kernel(const float* __restrict__ xqkv, int C, int q_off, int k_off, int v_off, const float* __restrict__ proj, int P,
                   int b_off, const float* __restrict__ a_raw, int A, int a_off, int dper, const float* __restrict__ dt_bias,
                   const float* __restrict__ a_log, const float* __restrict__ gate, int G, int z_off, int gate_kind,
@@ -1471,6 +1488,16 @@ delta_step_kernel(const float* __restrict__ xqkv, int C, int q_off, int k_off, i
     const float* ar = a_raw + t * A + a_off + (size_t)h * dper;
     const float* br = dt_bias + (size_t)h * dper;
     float* S = state + (size_t)slots[t] * slot_stride + (size_t)h * dv * dk;
+    float sv[RPL][DELTA_STEP_COLS];    // a group of columns' state: the first one is asked for before anything else
+    auto load = [&](int c0) {
+#pragma unroll
+        for (int i = 0; i < RPL; ++i) {
+            const int r = lane + 32 * i;
+#pragma unroll
+            for (int j = 0; j < DELTA_STEP_COLS; ++j) sv[i][j] = (r < dk && c0 + j < dv) ? S[(size_t)(c0 + j) * dk + r] : 0.f;
+        }
+    };
+    load(warp * DELTA_STEP_COLS);
     const float rate = expf(a_log[h]), beta = 1.0f / (1.0f + expf(-proj[t * P + b_off + h]));
     float kv[RPL], qv[RPL], gv[RPL];   // every warp has the head's key, query and decays in registers
     float ssk = 0.f, ssq = 0.f;
@@ -1503,13 +1530,9 @@ delta_step_kernel(const float* __restrict__ xqkv, int C, int q_off, int k_off, i
     }
     kq = tq_warp_sum(kq);
     for (int c0 = warp * DELTA_STEP_COLS; c0 < dv; c0 += n_warps * DELTA_STEP_COLS) {
-        float sv[RPL][DELTA_STEP_COLS], pred[DELTA_STEP_COLS], rd[DELTA_STEP_COLS];
+        float pred[DELTA_STEP_COLS], rd[DELTA_STEP_COLS], vc[DELTA_STEP_COLS];
 #pragma unroll
-        for (int i = 0; i < RPL; ++i) {
-            const int r = lane + 32 * i;
-#pragma unroll
-            for (int j = 0; j < DELTA_STEP_COLS; ++j) sv[i][j] = (r < dk && c0 + j < dv) ? S[(size_t)(c0 + j) * dk + r] : 0.f;
-        }
+        for (int j = 0; j < DELTA_STEP_COLS; ++j) vc[j] = c0 + j < dv ? vr[c0 + j] : 0.f;
 #pragma unroll
         for (int j = 0; j < DELTA_STEP_COLS; ++j) pred[j] = rd[j] = 0.f;
 #pragma unroll
@@ -1529,7 +1552,7 @@ delta_step_kernel(const float* __restrict__ xqkv, int C, int q_off, int k_off, i
 #pragma unroll
         for (int j = 0; j < DELTA_STEP_COLS; ++j) {
             if (c0 + j < dv) {
-                const float u = beta * (vr[c0 + j] - pred[j]);
+                const float u = beta * (vc[j] - pred[j]);
 #pragma unroll
                 for (int i = 0; i < RPL; ++i) {
                     const int r = lane + 32 * i;
@@ -1538,6 +1561,7 @@ delta_step_kernel(const float* __restrict__ xqkv, int C, int q_off, int k_off, i
                 if (lane == 0) s_o[c0 + j] = rd[j] + kq * u;
             }
         }
+        load(c0 + n_warps * DELTA_STEP_COLS);          // beyond dv: zeros, nothing is read
     }
     __syncthreads();
     float ss = 0.f;
@@ -1567,7 +1591,7 @@ TQ_EXPORT int tq_delta_step(const float* xqkv, int C, int q_off, int k_off, int 
     TQ_REQUIRE(b_off >= 0 && b_off + heads <= P && a_off >= 0 && a_off + heads * dper <= A && z_off >= 0 && z_off + heads * dv <= G,
                "delta_step: betas, decays or gates lie outside their rows");
     const int groups = (dv + DELTA_STEP_COLS - 1) / DELTA_STEP_COLS;                  // a warp a group, up to sixteen
-    const int threads = 32 * (groups >= 16 ? 16 : (groups >= 8 ? 8 : (groups >= 4 ? 4 : (groups >= 2 ? 2 : 1))));
+    const int threads = 32 * step_warps((long long)T_ * heads, groups);
 #define DELTA_STEP_LAUNCH(R)                                                                                            \
     TQ_DISPATCH(w_dtype, TW, TQ_DISPATCH(out_dtype, TO,                                                                 \
         (tq_launch(dim3(T_, heads), threads, (size_t)dv * sizeof(float), stream)(delta_step_kernel<R, TW, TO>, xqkv, C, q_off, k_off, v_off, \
