@@ -62,7 +62,7 @@ CONFIGS = {
                  layer("parallel", parallel(), ff=56),
                  layer("mlstm", memory(heads=2, dim=20, vdim=6, gate_cap=4.0), ff=24),
                  layer("parallel", parallel(left(heads=3, kv_heads=1, dim=10, vdim=6, temp=None), right(heads=2, kv_heads=2, dim=16, vdim=8, conv=2),
-                                            (-0.6, 0.9)), ff=32)]),
+                                            (-0.7, 1.1)), ff=32)]),
     # sizes the tensor-core attention kernels take (32 / 64 / 128), side by side first, one and several query heads a
     # key/value head, whole heads rotated, factors that the design could make equal or one
     "b": config([layer("parallel", parallel(left(heads=4, kv_heads=1, dim=64, vdim=32, scale=0.2, temp=(0.3, 64)),

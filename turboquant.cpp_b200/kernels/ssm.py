@@ -1,4 +1,5 @@
-"""Launchers of csrc/ssm.cu: the short causal convolution and the recurrence of a state-space mixer."""
+"""Launchers of csrc/ssm.cu: the short causal convolution, and the recurrences with a state per head (state-space mixer,
+retention, matrix memory, delta rules)."""
 from __future__ import annotations
 
 from ctypes import c_float, c_int, c_longlong
